@@ -9,13 +9,15 @@ required at import time; there is no CPU or PyTorch fallback.
 """
 
 from . import _lib  # noqa: F401  (raises if the shared object is missing)
-from .model.engine import Engine
+from .model.delunex import Delunex
+from .model.engine import Engine, StepRunner
 from .model.gpt import GPT, BaseGPT
-from .model.kv_cache import KVCache, PagedKVCache
+from .model.kv_cache import KVCache, LatentCache, PagedKVCache
+from .model.registry import load_model
 from .sampler.nucleus import NucleusSampler
 from .sampler.sampler import Sampler
 from .sampler.temperature import TemperatureSampler
 
 __all__ = [
-    "GPT", "BaseGPT", "KVCache", "PagedKVCache", "Engine", "Sampler", "TemperatureSampler", "NucleusSampler",
+    "GPT", "BaseGPT", "Delunex", "KVCache", "LatentCache", "PagedKVCache", "Engine", "StepRunner", "load_model", "Sampler", "TemperatureSampler", "NucleusSampler",
 ]

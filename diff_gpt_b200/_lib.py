@@ -88,10 +88,27 @@ PROTOTYPES = {
         [_p, _i64, _p, _i64, _f32, _f32, _f32, _u64, _i64, _p, _i32, _p, _p, _i32, _i64, _p, _p, _p, _p, _i64, _p, _i64, _p,
          _sz, _i32, _i32, _i32, _i32, _p, _p],
     ),
+    "dgpt_fmha_window": (
+        C.c_int,
+        [_p, _i64, _i64, _p, _p, _i64, _i64, _i64, _i32, _p, _i64, _i64, _p, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _f32,
+         _i32, _i32, _p, _p],
+    ),
+    "dgpt_latent_append": (C.c_int, [_p, _i64, _p, _f32, _i32, _kvp, _p, _p, _i32, _i32, _i32, _p, _i32, _p, _p]),
+    "dgpt_latent_attn_workspace_bytes": (_sz, [_i32, _i32, _i32, _i32]),
+    "dgpt_latent_attn": (
+        C.c_int,
+        [_p, _i64, _kvp, _p, _p, _p, _p, _p, _i64, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32, _p],
+    ),
+    "dgpt_embed_scale": (C.c_int, [_p, _p, _p, _i64, _i32, _i32, _f32, _i32, _p]),
+    "dgpt_norm_add": (C.c_int, [_p, _p, _f32, _p, _p, _p, _i64, _i32, _i32, _p]),
+    "dgpt_depth_avg_conv": (C.c_int, [_p, _i64, _i32, _p, _p, _i32, _p, _p, _p, _p, _i32, _i32, _i32, _i32, _p]),
+    "dgpt_layer_tail": (C.c_int, [_p, _p, _f32, _p, _p, _i64, _i32, _p, _p, _i32, _p, _p, _p, _i64, _i32, _i32, _p]),
+    "dgpt_depth_avg_norm": (C.c_int, [_p, _i64, _i32, _p, _p, _f32, _p, _p, _i64, _i64, _i32, _i32, _p]),
+    "dgpt_xielu": (C.c_int, [_p, _p, _i64, _f32, _f32, _i32, _p]),
 }
 _NOT_LAUNCHING = {
     "dgpt_last_error", "dgpt_version", "dgpt_decode_attn_workspace_bytes", "dgpt_decode_attn_static_capacity_bytes",
-    "dgpt_lmhead_workspace_bytes",
+    "dgpt_lmhead_workspace_bytes", "dgpt_latent_attn_workspace_bytes",
 }
 
 

@@ -171,6 +171,7 @@ struct KvView {
   int page_tokens;
   int max_pages;
   long long n_pages;  // pages addressable through the table (0 = not stated)
+  long long token_stride;  // elements between consecutive tokens of a head (0 = head_dim)
 };
 
 inline KvView make_view(const dgpt_kv_layout* l) {
@@ -183,6 +184,7 @@ inline KvView make_view(const dgpt_kv_layout* l) {
   w.page_tokens = l->page_tokens;
   w.max_pages = l->max_pages;
   w.n_pages = l->page_table ? l->n_pages : 0;
+  w.token_stride = 0;
   return w;
 }
 
@@ -192,7 +194,7 @@ __device__ __forceinline__ long long kv_offset(const KvView& kv, int seq, int he
   const int in = slot - lp * kv.page_tokens;
   const long long pg = kv.page_table ? (long long)kv.page_table[(long long)seq * kv.max_pages + lp]
                                      : (long long)seq;
-  return pg * kv.page_stride + (long long)head * kv.head_stride + (long long)in * D;
+  return pg * kv.page_stride + (long long)head * kv.head_stride + (long long)in * (kv.token_stride ? kv.token_stride : D);
 }
 
 inline int validate_kv(const dgpt_kv_layout* kv, int D) {

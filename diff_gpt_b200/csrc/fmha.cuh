@@ -19,6 +19,12 @@ struct FmhaArgs {
   int max_ctas;  // two-CTAs-per-SM kernel only: at most this many CTAs, looping over the query tiles (0 = one CTA per tile)
   int two_cta;  // tensor-core path only: the 128-thread kernel with two CTAs per SM instead of the warp-specialised one
   int pingpong;  // tensor-core path only: the kernel with two query tiles per CTA
+  // sliding-window form (dgpt_fmha_window); the defaults leave the kernels as dgpt_fmha_prefill uses them
+  int window = 0;           // query i sees keys (q_offset + i - window, q_offset + i]; 0 = all of them (causal only)
+  float scale = 0.f;        // score scale; 0 = 1 / sqrt(D)
+  long long kv_ts = 0;      // elements between consecutive keys of a head; 0 = D
+  const void* hgate = nullptr;  // [B * Tq, H] in dtype: output of head h is multiplied by sigmoid(hgate)
+  long long hgate_rs = 0;
 };
 
 // What the tensor-core kernels need besides the three tensor maps.
@@ -38,8 +44,22 @@ struct TcParams {
   int n_qt, n_work;  // query tiles per (batch, head) and work items in all (a capped grid loops over them)
   int d_head;        // head_dim of the tensors in global memory (32 rides on the 64-wide kernels: the TMA boxes are 64 wide
                      // and the columns past the tensor's extent arrive as zeros, so scores and outputs are unchanged)
+  int window;        // 0 = no lower bound
+  const void* hgate; // bf16 [B * Tq, H], or NULL
+  long long hgate_rs;
   int BH, group_bh;  // two-query-tile kernel: (batch, head) pairs in all, and how many are worked on at a time
 };
+
+// Factor that the per-head output gate puts on row `row` (b * Tq + i) of head h.
+template <typename T>
+__device__ __forceinline__ float head_gate(const void* hgate, long long rs, long long row, int h) {
+  if (hgate == nullptr) return 1.f;
+  return 1.f / (1.f + expf(-Io<T>::ld(static_cast<const T*>(hgate) + row * rs + h)));
+}
+// First key tile of `tile` keys that a query at position `first_q` (the tile's lowest) can see.
+__device__ __forceinline__ int window_first_tile(int window, int first_q, int tile) {
+  return window > 0 ? max(0, first_q - window + 1) / tile : 0;
+}
 
 // warp-level kernel (fmha_simt.cu)
 int fmha_simt(const FmhaArgs& a, const KvView& kv, cudaStream_t st);

@@ -19,7 +19,8 @@ template <typename T, int D, int SPLIT>
 __global__ void __launch_bounds__(128)
 fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView kv, const int* __restrict__ kv_len,
                  int kv_len_all, void* __restrict__ o, long long o_bs, long long o_rs, int o_f32,
-                 float* __restrict__ lse, int H, int Tq, int q_offset, int causal, float scale_log2) {
+                 float* __restrict__ lse, int H, int Tq, int q_offset, int causal, float scale_log2, int window,
+                 const void* __restrict__ hgate, long long hgate_rs) {
   constexpr int DP = D / SPLIT;       // elements per thread
   constexpr int BM = 128 / SPLIT;     // queries per CTA
   constexpr int VEC = Io<T>::kVec16;
@@ -36,6 +37,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
   int kmax = klen;
   if (causal) kmax = min(klen, q_offset + min(q0 + BM, Tq));
   const int my_last = causal ? q_offset + qi : 0x7fffffff;  // last visible key of this query
+  const int my_first = window > 0 ? q_offset + qi - window + 1 : 0;
 
   float qf[DP], acc[DP];
 #pragma unroll
@@ -57,7 +59,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
   const T* kbase = static_cast<const T*>(kv.k);
   const T* vbase = static_cast<const T*>(kv.v);
 
-  for (int j0 = 0; j0 < kmax; j0 += kSimtBN) {
+  for (int j0 = window_first_tile(window, q_offset + q0, kSimtBN) * kSimtBN; j0 < kmax; j0 += kSimtBN) {
     __syncthreads();
     constexpr int VPR = D / VEC;  // 16-byte vectors per key row
     for (int idx = tid; idx < kSimtBN * VPR; idx += 128) {
@@ -95,7 +97,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
 #pragma unroll
         for (int x = 1; x < SPLIT; x <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, x);
         const int j = j0 + kb + kk;
-        s[kk] = (q_ok && j < klen && j <= my_last) ? dot : -INFINITY;
+        s[kk] = (q_ok && j < klen && j <= my_last && j >= my_first) ? dot : -INFINITY;
         smax = fmaxf(smax, s[kk]);
       }
       if (smax == -INFINITY) continue;  // nothing visible in this group (no shuffles below)
@@ -122,7 +124,8 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
     }
   }
   if (!q_ok) return;
-  const float inv = l > 0.f ? 1.f / l : 0.f;
+  float inv = l > 0.f ? 1.f / l : 0.f;
+  inv *= head_gate<T>(hgate, hgate_rs, (long long)b * Tq + qi, h);
   const long long oo = (long long)b * o_bs + (long long)qi * o_rs + (long long)h * D + part * DP;
   if (o_f32) {
     float* op = static_cast<float*>(o) + oo;
@@ -144,10 +147,10 @@ static int fmha_simt_launch(const FmhaArgs& a, const KvView& kv, cudaStream_t st
   constexpr int SPLIT = D > 64 ? D / 64 : 1;
   constexpr int BM = 128 / SPLIT;
   dim3 grid((unsigned)((a.Tq + BM - 1) / BM), (unsigned)a.H, (unsigned)a.B);
-  const float scale_log2 = kLog2e / sqrtf((float)D);
+  const float scale_log2 = a.scale > 0.f ? a.scale * kLog2e : kLog2e / sqrtf((float)D);
   fmha_simt_kernel<T, D, SPLIT><<<grid, 128, 0, st>>>(static_cast<const T*>(a.q), a.q_bs, a.q_rs, kv, a.kv_len,
                                                       a.kv_len_all, a.o, a.o_bs, a.o_rs, a.o_f32, a.lse, a.H, a.Tq,
-                                                      a.q_offset, a.causal, scale_log2);
+                                                      a.q_offset, a.causal, scale_log2, a.window, a.hgate, a.hgate_rs);
   return launch_status("fmha_simt");
 }
 
@@ -216,5 +219,49 @@ extern "C" int dgpt_fmha_prefill(const void* q, int64_t q_batch_stride, int64_t 
     return DGPT_E_UNSUPPORTED;
   }
   if (tc_ok && impl != 1) return fmha_tc(a, *kv, st);
+  return fmha_simt(a, view, st);
+}
+
+extern "C" int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const void* k, const void* v,
+                                int64_t kv_batch_stride, int64_t kv_row_stride, int64_t kv_head_stride, int32_t n_keys, void* o,
+                                int64_t o_batch_stride, int64_t o_row_stride, const void* gate, int64_t gate_row_stride,
+                                int32_t B, int32_t H, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, float scale,
+                                int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(q && k && v && o, "fmha_window: NULL pointer");
+  DGPT_REQUIRE(B >= 0 && H > 0 && Tq >= 0 && B <= 65535 && H <= 65535 && n_keys >= 0, "fmha_window: bad sizes");
+  DGPT_REQUIRE(window >= 0 && q_offset >= 0 && scale > 0.f, "fmha_window: bad window, offset or scale");
+  DGPT_REQUIRE(q_row_stride % 8 == 0 && q_batch_stride % 8 == 0 && o_row_stride % 8 == 0 && o_batch_stride % 8 == 0 &&
+                   kv_batch_stride % 8 == 0 && kv_row_stride % 8 == 0 && kv_head_stride % 8 == 0,
+               "fmha_window: strides must be multiples of 8 elements");
+  DGPT_REQUIRE(impl >= 0 && impl <= 3, "fmha_window: impl must be 0 (auto), 1 (warp-level), 2 or 3 (tensor-core)");
+  if (B == 0 || Tq == 0) return DGPT_OK;
+  dgpt_kv_layout kv = {};
+  kv.k_base = const_cast<void*>(k);
+  kv.v_base = const_cast<void*>(v);
+  kv.page_stride = kv_batch_stride;
+  kv.head_stride = kv_head_stride;
+  kv.page_tokens = n_keys > 0 ? n_keys : 1;
+  if (int e = validate_kv(&kv, D)) return e;
+  FmhaArgs a;
+  a.q = q; a.q_bs = q_batch_stride; a.q_rs = q_row_stride;
+  a.kv_len = nullptr; a.kv_len_all = n_keys;
+  a.o = o; a.o_bs = o_batch_stride; a.o_rs = o_row_stride; a.o_f32 = 0; a.lse = nullptr;
+  a.B = B; a.H = H; a.Tq = Tq; a.D = D; a.q_offset = q_offset; a.causal = 1; a.dtype = dtype;
+  a.status = status;
+  a.max_ctas = 0;
+  a.pingpong = 0;
+  a.window = window; a.scale = scale; a.kv_ts = kv_row_stride;
+  a.hgate = gate; a.hgate_rs = gate_row_stride;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  // the persistent kernel from 1024 keys on, as for full attention; the keys a query tile meets are at most the window's
+  a.two_cta = impl == 3 || (impl == 0 && n_keys < 1024);
+  const bool tc_ok = fmha_tc_supported(a, kv);
+  if (impl >= 2 && !tc_ok) {
+    set_error("fmha_window: the tensor-core kernels do not cover dtype %d, head_dim %d with this layout", dtype, D);
+    return DGPT_E_UNSUPPORTED;
+  }
+  if (tc_ok && impl != 1) return fmha_tc(a, kv, st);
+  KvView view = make_view(&kv);
+  view.token_stride = kv_row_stride;
   return fmha_simt(a, view, st);
 }

@@ -91,11 +91,12 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
   const int q0 = qt * kBM;
   const int klen = p.kv_len ? p.kv_len[b] : p.kv_len_all;
   const int kmax = p.causal ? min(klen, p.q_offset + min(q0 + kBM, p.Tq)) : klen;
-  const int n_tiles = kmax > 0 ? (kmax + kBN - 1) / kBN : 0;
+  const int tile0 = window_first_tile(p.window, p.q_offset + q0, kBN);
+  const int n_tiles = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0);
 
   // Issue the TMA loads of key/value tile j (thread 0 only).  One box per page and per 64-wide half.
   auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t bar, int j) {
-    const int t0 = j * kBN;
+    const int t0 = (tile0 + j) * kBN;
     if (pt >= kBN) {
       const int lp = t0 / pt, in = t0 - lp * pt;
       const int pg = p.page_table ? p.page_table[(long long)b * p.max_pages + lp] : b;
@@ -129,7 +130,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
 
   for (int j = 0; j < n_tiles; ++j) {
     const uint32_t par = (uint32_t)(j & 1);
-    const int t0 = j * kBN;
+    const int t0 = (tile0 + j) * kBN;
     // ---- S = Q K^T ----
     if (tid == 0) {
       bool ok = true;
@@ -172,8 +173,10 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
       fence_async_smem();
     }
     // ---- softmax of this row ----
-    const bool need_mask = (t0 + kBN > klen) || (p.causal && t0 + kBN - 1 > p.q_offset + q0);
+    const bool need_mask = (t0 + kBN > klen) || (p.causal && t0 + kBN - 1 > p.q_offset + q0) ||
+                           (p.window > 0 && t0 <= p.q_offset + q0 + kBM - 1 - p.window);
     const int last_key = p.causal ? min(klen - 1, p.q_offset + q0 + tid) : klen - 1;
+    const int first_key = p.window > 0 ? p.q_offset + q0 + tid - p.window + 1 : 0;
     float sv[kBN];
 #pragma unroll
     for (int c = 0; c < 4; ++c) tmem_ld32_nowait(lane_addr + c * 32, &sv[c * 32]);
@@ -182,7 +185,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
     if (need_mask) {
 #pragma unroll
       for (int i = 0; i < kBN; ++i) {
-        sv[i] = (t0 + i <= last_key) ? sv[i] : -INFINITY;
+        sv[i] = (t0 + i <= last_key && t0 + i >= first_key) ? sv[i] : -INFINITY;
         mx = fmaxf(mx, sv[i]);
       }
     } else {
@@ -259,7 +262,8 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
     // tcgen05.ld is warp-collective: every thread reads its row, only rows that exist are stored
     const int qi = q0 + tid;
     const bool row_ok = qi < p.Tq;
-    const float inv = (l > 0.f && n_tiles > 0) ? 1.f / l : 0.f;
+    float inv = (l > 0.f && n_tiles > 0) ? 1.f / l : 0.f;
+    if (p.hgate && row_ok) inv *= head_gate<__nv_bfloat16>(p.hgate, p.hgate_rs, (long long)b * p.Tq + qi, h);
     const long long off = (long long)b * p.o_bs + (long long)qi * p.o_rs + (long long)h * p.d_head;
 #pragma unroll
     for (int c = 0; c < D / 32; ++c) {
@@ -307,8 +311,11 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
 bool fmha_tc_supported(const FmhaArgs& a, const dgpt_kv_layout& kv) {
   if (a.dtype != DGPT_BF16 || (a.D != 32 && a.D != 64 && a.D != 128)) return false;
   const int pt = kv.page_tokens;
-  if (!((pt >= tc::kBN && pt % tc::kBN == 0) || (pt >= 8 && pt < tc::kBN && tc::kBN % pt == 0))) return false;
-  if (kv.page_table == nullptr && pt < tc::kBN) return false;
+  // One dense run of keys per sequence with a stated token stride (dgpt_fmha_window) may have any length: a tile never
+  // leaves the run's tensor, and what the box covers past its end arrives as zeros.
+  const bool run = a.kv_ts > 0 && kv.page_table == nullptr;
+  if (!run && !((pt >= tc::kBN && pt % tc::kBN == 0) || (pt >= 8 && pt < tc::kBN && tc::kBN % pt == 0))) return false;
+  if (!run && kv.page_table == nullptr && pt < tc::kBN) return false;
   auto al16 = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   if (!al16(a.q) || !al16(a.o) || !al16(kv.k_base) || !al16(kv.v_base)) return false;
   if (a.q_rs % 8 || a.q_bs % 8 || a.o_rs % 8 || a.o_bs % 8 || kv.head_stride % 8 || kv.page_stride % 8) return false;
@@ -335,8 +342,9 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
     const int pt = kv.page_tokens;
     cuuint64_t n_pages = kv.page_table ? (kv.n_pages > 0 ? (cuuint64_t)kv.n_pages : (cuuint64_t)1 << 24) : (cuuint64_t)a.B;
     const cuuint64_t dims[4] = {(cuuint64_t)d_head, (cuuint64_t)pt, (cuuint64_t)a.H, n_pages};
-    const cuuint64_t strides[3] = {(cuuint64_t)d_head * 2, (cuuint64_t)kv.head_stride * 2, (cuuint64_t)kv.page_stride * 2};
-    const cuuint32_t box[4] = {64, (cuuint32_t)(pt < kBN ? pt : kBN), 1, 1};
+    const cuuint64_t strides[3] = {(cuuint64_t)(a.kv_ts > 0 ? a.kv_ts : d_head) * 2, (cuuint64_t)kv.head_stride * 2,
+                                   (cuuint64_t)kv.page_stride * 2};
+    const cuuint32_t box[4] = {64, (cuuint32_t)(pt < kBN && a.kv_ts == 0 ? pt : kBN), 1, 1};
     if (!encode_map(&mk, kv.k_base, dims, strides, box)) return DGPT_E_CUDA;
     if (!encode_map(&mv, kv.v_base, dims, strides, box)) return DGPT_E_CUDA;
   }
@@ -345,7 +353,7 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   p.kv_len_all = a.kv_len_all;
   p.page_table = kv.page_table;
   p.max_pages = kv.max_pages;
-  p.page_tokens = kv.page_tokens;
+  p.page_tokens = a.kv_ts > 0 ? (kv.page_tokens + kBN - 1) / kBN * kBN : kv.page_tokens;  // a run is one page of whole tiles
   p.o = a.o;
   p.o_bs = a.o_bs;
   p.o_rs = a.o_rs;
@@ -355,7 +363,10 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   p.Tq = a.Tq;
   p.q_offset = a.q_offset;
   p.causal = a.causal;
-  p.scale_log2 = kLog2e / sqrtf((float)d_head);
+  p.scale_log2 = a.scale > 0.f ? a.scale * kLog2e : kLog2e / sqrtf((float)d_head);
+  p.window = a.window;
+  p.hgate = a.hgate;
+  p.hgate_rs = a.hgate_rs;
   p.d_head = d_head;
   p.status = a.status;
   p.n_qt = (a.Tq + kBM - 1) / kBM;

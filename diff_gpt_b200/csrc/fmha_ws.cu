@@ -35,7 +35,7 @@ constexpr int kWsThreads = 320;  // 8 softmax warps, the MMA issuer's warp, the 
 constexpr uint32_t kWsTmemCols = 512;
 
 struct WsItem {
-  int b, h, q0, klen, n;  // n = key tiles
+  int b, h, q0, klen, tile0, n;  // n = key tiles, the first of them tile0 (0 unless a sliding window cuts the rest off)
 };
 
 __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
@@ -45,7 +45,8 @@ __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
   it.q0 = qt * kBM;
   it.klen = p.kv_len ? p.kv_len[it.b] : p.kv_len_all;
   const int kmax = p.causal ? min(it.klen, p.q_offset + min(it.q0 + kBM, p.Tq)) : it.klen;
-  it.n = kmax > 0 ? (kmax + kBN - 1) / kBN : 0;
+  it.tile0 = window_first_tile(p.window, p.q_offset + it.q0, kBN);
+  it.n = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0);
   return it;
 }
 
@@ -118,7 +119,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         const WsItem it = ws_item(p, bh, qt);
         if (it.n == 0) continue;
         auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t full, int j) {
-          const int t0 = j * kBN;
+          const int t0 = (it.tile0 + j) * kBN;
           if (pt >= kBN) {
             const int lp = t0 / pt, in = t0 - lp * pt;
             const int pg = p.page_table ? p.page_table[(long long)it.b * p.max_pages + lp] : it.b;
@@ -264,7 +265,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       float m = -INFINITY, l = 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const unsigned g = g0 + (unsigned)j, buf = g & 1u, ph = (g >> 1) & 1u;
-        const int t0 = j * kBN;
+        const int t0 = (it.tile0 + j) * kBN;
         // exits are taken by whole warps (the vote makes the decision uniform), never by single lanes
         if (!__all_sync(0xffffffffu, wait_or_abort(bar_s0 + 8 * buf, ph, abort_flag, 23))) {
           fail = true;
@@ -287,8 +288,10 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
             fence_async_smem();
           }
         }
-        const bool need_mask = (t0 + kBN > klen) || (p.causal && t0 + kBN - 1 > p.q_offset + q0);
+        const bool need_mask = (t0 + kBN > klen) || (p.causal && t0 + kBN - 1 > p.q_offset + q0) ||
+                               (p.window > 0 && t0 <= p.q_offset + q0 + kBM - 1 - p.window);
         const int last_key = p.causal ? min(klen - 1, p.q_offset + q0 + row) : klen - 1;
+        const int first_key = p.window > 0 ? p.q_offset + q0 + row - p.window + 1 : 0;
         const int c0 = t0 + half * kHalf;  // key index of this thread's first column
         float sv[kHalf];
 #pragma unroll
@@ -296,7 +299,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         tc_wait_ld();
         if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key) ? sv[i] : -INFINITY;
+          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key && c0 + i >= first_key) ? sv[i] : -INFINITY;
         }
         // One sweep turns this thread's 64 scores into probabilities against a reference maximum `ref` (log2 domain),
         // writes them as packed bf16 into the P buffer and returns their sum.
@@ -404,7 +407,8 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       }
       const int qi = q0 + row;
       const bool row_ok = qi < p.Tq;
-      const float inv = (l > 0.f && n_tiles > 0) ? 1.f / l : 0.f;
+      float inv = (l > 0.f && n_tiles > 0) ? 1.f / l : 0.f;
+      if (p.hgate && row_ok) inv *= head_gate<__nv_bfloat16>(p.hgate, p.hgate_rs, (long long)b * p.Tq + qi, h);
       const long long off = (long long)b * p.o_bs + (long long)qi * p.o_rs + (long long)h * p.d_head + half * (D / 2);
 #pragma unroll
       for (int c = 0; c < D / 64; ++c) {

@@ -5,6 +5,7 @@
 //   mode 0:  out[m, n]     = bf16(acc[m, n])
 //   mode 1:  out[m, n / 2] = swiglu(bf16(acc[m, n]), bf16(acc[m, n + 1]))   for even n  (interleaved gate / linear)
 //   mode 2:  out[m, n]     = bf16(resid[m, n] + acc[m, n])                    (the residual add of addmm, one rounding)
+//   mode 4:  out[m, n]     = bf16(xielu(acc[m, n]))   with alpha_p = alpha, alpha_n = limit
 //   mode 3:  nothing is stored: row m keeps the best key of  key[m, n] = cap(bf16(acc[m, n])) / T + Gumbel noise(m, n)
 //            (no noise and T = 1 for an arg-max) in best[m], a 64-bit word (order-preserving key bits, ~n) raised with
 //            atomicMax - the tied-embedding head with the draw in its epilogue, so [M, N] logits never reach HBM
@@ -22,6 +23,7 @@
 // fill 148 SMs evenly and no overlapped epilogue - 30.7 us.
 // Every mbarrier wait is bounded; a wait that runs out raises a CTA-wide abort flag, is reported through
 // the status word, and every role drains what it issued before TMEM is freed.
+#include "activation.cuh"
 #include "linear.cuh"
 #include "sampling.cuh"
 #include "tcgen05.cuh"
@@ -223,7 +225,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ C
           continue;
         }
         if (DRAW) continue;
-        if (p.mode == 0 || p.mode == 2) {
+        if (p.mode != 1) {
           __nv_bfloat16* dst = p.out + (long long)row * p.out_rs + col0 + c;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
@@ -233,6 +235,9 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ C
               ld16<__nv_bfloat16>(p.resid + (long long)row * p.resid_rs + col0 + c + 8 * q, r8);
 #pragma unroll
               for (int x = 0; x < 8; ++x) v[8 * q + x] += r8[x];
+            } else if (p.mode == 4) {
+#pragma unroll
+              for (int x = 0; x < 8; ++x) v[8 * q + x] = xielu_value(v[8 * q + x], p.alpha, p.limit);
             }
             st16<__nv_bfloat16>(dst + 8 * q, v + 8 * q, 1.f);
           }
@@ -329,7 +334,8 @@ int dgpt::linear_launch(const void* a, int64_t a_row_stride, const void* w, int6
                         const HeadDraw* draw, void* stream) {
   DGPT_REQUIRE(a && w && (out || epilogue == 3), "linear: NULL pointer");
   DGPT_REQUIRE(M >= 0 && N > 0 && K > 0, "linear: bad sizes");
-  DGPT_REQUIRE(epilogue >= 0 && epilogue <= 3, "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add) or 3 (draw)");
+  DGPT_REQUIRE(epilogue >= 0 && epilogue <= 4,
+               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add), 3 (draw) or 4 (xIELU)");
   DGPT_REQUIRE(epilogue != 2 || resid, "linear: epilogue 2 needs the matrix to add");
   DGPT_REQUIRE(epilogue != 3 || (draw && draw->best), "linear: epilogue 3 needs the draw parameters");
   if (dtype != DGPT_BF16) {
@@ -412,7 +418,8 @@ extern "C" int dgpt_linear(const void* a, int64_t a_row_stride, const void* w, i
                            int64_t out_row_stride, const void* resid, int64_t resid_row_stride, int32_t M, int32_t N,
                            int32_t K, int32_t epilogue, float alpha, float limit, int32_t dtype, int32_t* status,
                            void* stream) {
-  DGPT_REQUIRE(epilogue >= 0 && epilogue <= 2, "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs) or 2 (add)");
+  DGPT_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 4,
+               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add) or 4 (xIELU)");
   return linear_launch(a, a_row_stride, w, w_row_stride, out, out_row_stride, resid, resid_row_stride, M, N, K, epilogue, alpha,
                        limit, dtype, status, nullptr, stream);
 }

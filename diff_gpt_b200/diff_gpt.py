@@ -20,7 +20,7 @@ import torch
 
 from .encoder_decoder import decode, encode
 from .model.engine import Engine
-from .model.gpt import GPT, BaseGPT
+from .model.gpt import BaseGPT, DeviceModel
 from .sampler.sampler import Sampler
 
 
@@ -70,9 +70,9 @@ class DiffGPT:
         return int(arr.max())
 
     def _device_codec(self, n_cols: int) -> bool:
-        """True when values <-> tokens can run on the device: this package's GPT, and difference orders the device
+        """True when values <-> tokens can run on the device: a model of this package, and difference orders the device
         codec covers.  Higher orders take the host codec (any order), then the same device decode of the tokens."""
-        return isinstance(self.model, GPT) and self._max_order(n_cols, "columns") <= DEVICE_CODEC_MAX_ORDER
+        return isinstance(self.model, DeviceModel) and self._max_order(n_cols, "columns") <= DEVICE_CODEC_MAX_ORDER
 
     def _encode(self, values: np.ndarray):
         return encode(
@@ -119,7 +119,7 @@ class DiffGPT:
         assert not self.use_decimal, "the Decimal code path of the reference codec is not part of this build"
         assert values.dtype == np.float64 and values.ndim == 3
         columns = values.shape[2]
-        dev = self.model.token_embedding_table.weight.device
+        dev = self.model.embedding.device
         orders = _orders(self.order_of_derivative, columns)
         scale = torch.from_numpy(column_scales(self.model.vocab_size, self.domain_of_definition, orders)).to(dev)
         orders_dev = torch.from_numpy(orders.astype(np.int32)).to(dev)
@@ -156,7 +156,7 @@ class DiffGPT:
         """`predict_samples` for several equally shaped frames in one decode: (S, num_samples, max_new_points, F).
         The reference loops over series on the host (benchmarks/prob_m4_bench.py:174-182).  Trajectory n of
         series s draws the random stream keyed by (s, n); `predict_samples` is the case S = 1."""
-        assert isinstance(self.model, GPT), "predict_samples_many needs the diff_gpt_b200 GPT"
+        assert isinstance(self.model, DeviceModel), "predict_samples_many needs a model of this package"
         assert len(dfs) > 0
         assert self._device_codec(dfs[0].shape[1]), f"difference orders above {DEVICE_CODEC_MAX_ORDER}: call predict_samples per frame"
         shape = dfs[0].shape

@@ -29,8 +29,8 @@ import torch.distributed as dist
 
 from .. import _lib, ops
 from ..sampler.sampler import Sampler
-from .gpt import GPT, BaseGPT, ForwardPlan, KvBinding, _pick_splits  # noqa: F401
-from .kv_cache import KVCache, PagedKVCache
+from .gpt import BaseGPT, DeviceModel, _pick_splits  # noqa: F401
+from .kv_cache import KVCache
 
 SHARED_PREFIX_MIN_ROWS = 16  # below this the prompt is read by the per-row kernel (split along keys)
 
@@ -53,7 +53,7 @@ class DecodeRun:
     def key_for(model, prompt_lens, num_samples, max_tokens, sampler, seed, has_force, page_tokens, use_graph,
                 fmha_impl, overlap_prefix, shared_prefix=None, fused_head=True, prefill_shared=False) -> tuple:
         spec = (1.0, 1.0) if sampler is None else (sampler.native_spec() if isinstance(sampler, Sampler) else None)
-        emb = model.token_embedding_table.weight
+        emb = model.embedding
         return (
             id(model), str(emb.device), emb.dtype, tuple(prompt_lens), num_samples, max_tokens, spec,
             None if spec is not None else id(sampler), seed, has_force, page_tokens, use_graph, fmha_impl,
@@ -62,7 +62,7 @@ class DecodeRun:
 
     def __init__(
         self,
-        model: GPT,
+        model: DeviceModel,
         prompts: list[list[int]],
         num_samples: int,
         max_tokens: int,
@@ -81,15 +81,13 @@ class DecodeRun:
         prefill_group=None,
     ) -> None:
         self.model = model
-        emb = model.token_embedding_table.weight
+        emb = model.embedding
         if not emb.is_cuda:
             raise RuntimeError("diff_gpt_b200.Engine runs on CUDA only; there is no CPU path")
         dev, dt = emb.device, emb.dtype
         self.dev = dev
         S, N, G = len(prompts), num_samples, max_tokens
         self.S, self.N, self.G, self.R = S, N, G, S * N
-        H, L = model.n_head, model.n_layer
-        D = model.n_embd // H
         self.cap = float(model.logit_softcap)
         self.seed = seed
         self.use_graph = use_graph
@@ -107,9 +105,8 @@ class DecodeRun:
             overlap_prefix, shared_prefix, fused_head, prefill_group is not None,
         )
         self.packed = model.packed_weights()  # the graph holds these tensors' addresses
-        self.cache = PagedKVCache(L, H, D, S, N, max(lens), G, dt, dev, page_tokens=page_tokens, pool=kv_pool)
+        self.cache = model.paged_cache(S, N, max(lens), G, page_tokens, kv_pool)
         self.prefix_lens = torch.tensor(lens, dtype=torch.int32, device=dev)
-        row_len = self.prefix_lens.repeat_interleave(N)
         self.tokens = torch.zeros(self.R, dtype=torch.int32, device=dev)
         self.history = torch.zeros((self.R, max(G, 1)), dtype=torch.int32, device=dev)
         self.step = torch.zeros(1, dtype=torch.int32, device=dev)
@@ -124,7 +121,7 @@ class DecodeRun:
         # K/V.  With a process group each rank prefills a contiguous block of S / W series only and the ranks exchange
         # the prompt pages and the last-position logits with one all-gather each (NCCL; each rank's own memory only).
         self.prefill_group, self.prefill_world, self.prefill_rank = None, 1, 0
-        if prefill_group is not None and dist.is_available() and dist.is_initialized():
+        if prefill_group is not None and self.cache.prompts_exchangeable and dist.is_available() and dist.is_initialized():
             w = dist.get_world_size(prefill_group)
             if w > 1 and S % w == 0:
                 self.prefill_group, self.prefill_world, self.prefill_rank = prefill_group, w, dist.get_rank(prefill_group)
@@ -137,40 +134,15 @@ class DecodeRun:
         for s, n in enumerate(lens):
             if s in mine:
                 groups.setdefault(n, []).append(s)
-        zero = torch.zeros(S, dtype=torch.int32, device=dev)
         self.prefills = []
         for P, members in groups.items():
-            idx = torch.tensor(members, device=dev)
-            table = self.cache.prefix_table[idx].contiguous()
-            layouts = [self.cache._layout(l, table) for l in range(L)]
-            bind = KvBinding(
-                layouts=layouts, pos0=zero[: len(members)], slot0=zero[: len(members)], kv_len=P, q_offset=0,
-                fmha_impl=fmha_impl,
-            )
-            plan = ForwardPlan(model, len(members), P, last_only=True)
-            self.prefills.append((P, members, idx, bind, plan, table))
+            bind, plan = model.prefill_plan(self.cache, members, P, fmha_impl)
+            self.prefills.append((P, members, torch.tensor(members, device=dev), bind, plan))
 
         # ---- decode plan ----
         # A shard of a larger job takes the path the whole job would take (the two paths round differently), so the
         # caller may decide; by default the prompt is shared from SHARED_PREFIX_MIN_ROWS trajectories per series on.
         shared = (N >= SHARED_PREFIX_MIN_ROWS) if shared_prefix is None else bool(shared_prefix)
-        slot0 = torch.full((self.R,), self.cache.suffix_slot0, dtype=torch.int32, device=dev)
-        self.bind = KvBinding(
-            layouts=[self.cache.row_layout(l) for l in range(L)],
-            pos0=row_len.contiguous(),
-            slot0=slot0,
-            step=self.step,
-            decode=True,
-            len0=row_len.contiguous(),
-            start1=slot0,
-            len1=torch.ones(self.R, dtype=torch.int32, device=dev),
-            n_splits=1 if shared else _pick_splits(self.R * H, max(lens) + G),
-            shared_layouts=[self.cache.prefix_layout(l) for l in range(L)] if shared else None,
-            shared_len=self.prefix_lens if shared else None,
-            rows_per_series=N,
-            fmha_impl=fmha_impl,
-            overlap_prefix=overlap_prefix and shared,
-        )
         # The head of a decode step.  With one of the library's samplers and a bf16 model it is one call,
         # dgpt_lmhead_sample: without a top-p filter the logits are sampled inside the GEMM's epilogue and never
         # stored (`fused_head`); with one, or when a caller wants to see them, the GEMM writes them for the
@@ -185,7 +157,9 @@ class DecodeRun:
                 self.head_logits = torch.empty((self.R, V), dtype=dt, device=dev)
             else:
                 self.head_ws = torch.empty(max(1, ops.lmhead_workspace_bytes(self.R) // 8), dtype=torch.int64, device=dev)
-        self.plan = ForwardPlan(model, self.R, 1, want_logits=not self.lmhead)
+        self.bind, self.plan = model.decode_plan(
+            self.cache, self.prefix_lens, max(lens) + G, self.step, shared, fmha_impl, overlap_prefix, want_logits=not self.lmhead
+        )
         self.graph = None
         self.done = 0  # tokens produced so far per row
         self.rng = None
@@ -213,7 +187,8 @@ class DecodeRun:
             self.force.copy_(f)
         self.step.zero_()
         self.plan.status.zero_()
-        for P, members, idx, bind, plan, _table in self.prefills:
+        self.cache.begin_prompts()
+        for P, members, idx, bind, plan in self.prefills:
             if on_device:
                 ids32 = prompts.reshape(-1) if len(members) == S else prompts[idx].reshape(-1)
             else:
@@ -225,6 +200,7 @@ class DecodeRun:
                 self.logits0[idx] = out
         if self.prefill_group is not None:
             self._exchange_prompts()
+        self.cache.prompts_ready()
         self.done = 0
         self.rng = None
 
@@ -335,6 +311,7 @@ class DecodeRun:
                     workspace=self.head_ws, status=self.plan.status,
                 )
             ops.step_advance(self.step, 0)
+            self.cache.prompts_ready()  # whatever state the warm-up advanced goes back to the prompt's end
             torch.cuda.synchronize(self.dev)
             self.graph = torch.cuda.CUDAGraph()
             before = _lib.stats.launches
@@ -407,13 +384,13 @@ class Engine:
         decode different trajectories of these same prompts; each rank then prefills only its share of the prompts
         and the ranks exchange the prompt K/V (every rank of the group must make the call).
         """
-        assert isinstance(self.model, GPT), "generate_many needs the diff_gpt_b200 GPT"
+        assert isinstance(self.model, DeviceModel), "generate_many needs a model of this package"
         assert len(prompts) > 0 and all(len(p) > 0 for p in prompts), "tokens must be non-empty"
         if isinstance(prompts, torch.Tensor):
             assert prompts.is_cuda and prompts.dtype == torch.int32 and prompts.dim() == 2 and prompts.is_contiguous()
         G = min(_effective_max_tokens(self.model.block_size, len(p), max_tokens) for p in prompts)
         S = len(prompts)
-        dev = self.model.token_embedding_table.weight.device
+        dev = self.model.embedding.device
         if G == 0 or num_samples == 0:
             z = torch.zeros((S, num_samples, G), dtype=torch.int32, device=dev)
             return z, z.clone()
@@ -475,7 +452,7 @@ class Engine:
             assert len(force_schedule) >= G, (
                 f"force_schedule must cover all generation steps (len={len(force_schedule)} < {G})"
             )
-        if not isinstance(self.model, GPT):
+        if not isinstance(self.model, DeviceModel):
             yield from _generate_generic(self.model, tokens, num_samples, G, sampler, seed, force_schedule)
             return
         run = DecodeRun(
@@ -505,7 +482,7 @@ class Engine:
             raise TypeError(f"generate() got an unexpected keyword argument {sorted(unknown)[0]!r}")
         results = [list(tokens) for _ in range(num_samples)]
         masks = [[0] * len(tokens) for _ in range(num_samples)]
-        if isinstance(self.model, GPT) and isinstance(tokens, list) and len(tokens) > 0 and all(
+        if isinstance(self.model, DeviceModel) and isinstance(tokens, list) and len(tokens) > 0 and all(
             isinstance(t, int) for t in tokens
         ):
             sched = kwargs.get("force_schedule")
@@ -523,6 +500,41 @@ class Engine:
                 results[i].append(column[i])
                 masks[i].append(column_masks[i])
         return results, masks
+
+
+class StepRunner:
+    """Requests whose tokens are given, not sampled: each call of `step` runs a request's next tokens behind what its
+    cache holds, in portions of any size, and returns the logits at the places asked for.
+
+    Every request has a cache of its own; `finish` gives it back, and a later request takes it over.
+    """
+
+    def __init__(self, model: DeviceModel) -> None:
+        self.model = model
+        self._live: dict = {}
+        self._free: list = []
+
+    def _cache(self, request):
+        if request not in self._live:
+            cache = self._free.pop() if self._free else self.model.new_cache()
+            cache.reset()
+            self._live[request] = cache
+        return self._live[request]
+
+    @torch.inference_mode()
+    def step(self, request, tokens: list[int], want: list[int]) -> torch.Tensor:
+        """fp32 [len(want), V] on the device; `want` names places among `tokens`."""
+        assert len(tokens) > 0 and all(0 <= t < self.model.vocab_size for t in tokens), "tokens must be ids of the vocabulary"
+        assert all(0 <= w < len(tokens) for w in want), "wanted places must lie among the tokens of the step"
+        dev = self.model.embedding.device
+        idx = torch.tensor([tokens], dtype=torch.int64, device=dev)
+        rows = torch.tensor(want, dtype=torch.int64, device=dev)
+        return self.model.logits_at(idx, self._cache(request), rows).to(torch.float32, copy=True)
+
+    def finish(self, request) -> None:
+        cache = self._live.pop(request, None)
+        if cache is not None:
+            self._free.append(cache)
 
 
 def _generate_generic(model, tokens, num_samples, G, sampler, seed, force_schedule):

@@ -58,6 +58,45 @@ class BaseGPT(nn.Module, ABC):
         ...
 
 
+class DeviceModel(BaseGPT):
+    """A model whose forward is enqueued by a plan of this library's kernels: what the Engine, the step-by-step
+    runner and the facade need from it, whatever its layers are."""
+
+    logit_softcap: float = 0.0
+
+    @property
+    @abstractmethod
+    def embedding(self) -> torch.Tensor:
+        """The token table [V, C], which is also the output head; its device and dtype are the model's."""
+
+    @abstractmethod
+    def packed_weights(self):
+        """Weights as the kernels want them; the same object until a parameter is modified or moved."""
+
+    # -- requests fed step by step --
+    @abstractmethod
+    def new_cache(self, batch_size: int = 1, seq_len: int = 0):
+        """An empty cache with `reset()` and `get_pos()` for `forward(idx, kv_cache=...)`."""
+
+    @abstractmethod
+    def logits_at(self, idx: torch.Tensor, cache, rows: torch.Tensor) -> torch.Tensor:
+        """Run idx (1, T) behind what `cache` holds; the logits [len(rows), V] of the given places among the T tokens."""
+
+    # -- batched decode (DecodeRun) --
+    @abstractmethod
+    def paged_cache(self, n_series: int, rows_per_series: int, prefix_len: int, max_new: int, page_tokens: int, pool=None):
+        """The cache of a decode run: prompt pages shared by a series' rows, private pages per row."""
+
+    @abstractmethod
+    def prefill_plan(self, cache, members: list[int], P: int, fmha_impl: int):
+        """(binding, plan) that prefills the P-token prompts of the series `members` into `cache`."""
+
+    @abstractmethod
+    def decode_plan(self, cache, prompt_lens: torch.Tensor, max_keys: int, step: torch.Tensor, shared: bool, fmha_impl: int,
+                    overlap_prefix: bool, want_logits: bool):
+        """(binding, plan) of one decode step of all rows; `step` is the device counter of generated tokens."""
+
+
 # ---- parameter containers (names and shapes of the reference state_dict) -------
 class SwiGLU(nn.Module):
     def __init__(self, alpha: float, limit: float) -> None:
@@ -355,7 +394,7 @@ class _Packed:
     stamp: tuple
 
 
-class GPT(BaseGPT):
+class GPT(DeviceModel):
     def __init__(
         self,
         vocab_size: int,
@@ -426,6 +465,67 @@ class GPT(BaseGPT):
             table = self.freqs_cis.to(emb.dtype).contiguous()
         self._packed = _Packed(emb=emb, freqs_cis=table, layers=layers, stamp=stamp)
         return self._packed
+
+    @classmethod
+    def from_config(cls, config: dict) -> "GPT":
+        """The constructor's keywords as a configuration."""
+        return cls(**{k: v for k, v in config.items() if k != "architecture"})
+
+    def load_tensors(self, tensors: dict) -> None:
+        """A checkpoint under the state_dict names; the tied head may be left out."""
+        tensors = dict(tensors)
+        tensors.setdefault("lm_head.weight", tensors["token_embedding_table.weight"])
+        self.load_state_dict(tensors)
+
+    # ---- what the Engine needs ----------------------------------------------------------
+    @property
+    def embedding(self) -> torch.Tensor:
+        return self.token_embedding_table.weight
+
+    def new_cache(self, batch_size: int = 1, seq_len: int = 0) -> KVCache:
+        return KVCache(batch_size=batch_size, num_heads=self.n_head, seq_len=max(seq_len, 1),
+                       head_dim=self.n_embd // self.n_head, num_layers=self.n_layer)
+
+    @torch.inference_mode()
+    def logits_at(self, idx: torch.Tensor, cache: KVCache, rows: torch.Tensor) -> torch.Tensor:
+        return self(idx, kv_cache=cache)[0][0].index_select(0, rows)
+
+    def paged_cache(self, n_series, rows_per_series, prefix_len, max_new, page_tokens, pool=None) -> PagedKVCache:
+        emb = self.embedding
+        return PagedKVCache(self.n_layer, self.n_head, self.n_embd // self.n_head, n_series, rows_per_series, prefix_len, max_new,
+                            emb.dtype, emb.device, page_tokens=page_tokens, pool=pool)
+
+    def prefill_plan(self, cache, members, P, fmha_impl):
+        idx = torch.tensor(members, device=cache.prefix_table.device)
+        table = cache.prefix_table[idx].contiguous()
+        zero = torch.zeros(len(members), dtype=torch.int32, device=table.device)
+        bind = KvBinding(
+            layouts=[cache._layout(l, table) for l in range(self.n_layer)], pos0=zero, slot0=zero, kv_len=P, q_offset=0,
+            fmha_impl=fmha_impl,
+        )
+        return bind, ForwardPlan(self, len(members), P, last_only=True)
+
+    def decode_plan(self, cache, prompt_lens, max_keys, step, shared, fmha_impl, overlap_prefix, want_logits):
+        R, L = cache.n_rows, self.n_layer
+        row_len = prompt_lens.repeat_interleave(cache.rows_per_series)
+        slot0 = torch.full((R,), cache.suffix_slot0, dtype=torch.int32, device=row_len.device)
+        bind = KvBinding(
+            layouts=[cache.row_layout(l) for l in range(L)],
+            pos0=row_len.contiguous(),
+            slot0=slot0,
+            step=step,
+            decode=True,
+            len0=row_len.contiguous(),
+            start1=slot0,
+            len1=torch.ones(R, dtype=torch.int32, device=row_len.device),
+            n_splits=1 if shared else _pick_splits(R * self.n_head, max_keys),
+            shared_layouts=[cache.prefix_layout(l) for l in range(L)] if shared else None,
+            shared_len=prompt_lens if shared else None,
+            rows_per_series=cache.rows_per_series,
+            fmha_impl=fmha_impl,
+            overlap_prefix=overlap_prefix and shared,
+        )
+        return bind, ForwardPlan(self, R, 1, want_logits=want_logits)
 
     # ---- the reference contract --------------------------------------------------------
     def forward(

@@ -146,6 +146,14 @@ class PagedKVCache:
     def bytes(self) -> int:
         return self.pool.numel() * self.pool.element_size()
 
+    prompts_exchangeable = True  # the prompt pages of a block of series are one run of the pool
+
+    def begin_prompts(self) -> None:
+        """Called before a new set of prompts is prefilled."""
+
+    def prompts_ready(self) -> None:
+        """Called when every prompt is in place, and again to undo a decode forward that was only a warm-up."""
+
     def _layout(self, layer: int, table: torch.Tensor) -> ops.KvLayout:
         H, pt, D = self.n_head, self.page_tokens, self.head_dim
         p = self.pool[layer]
@@ -161,3 +169,153 @@ class PagedKVCache:
     def row_layout(self, layer: int) -> ops.KvLayout:
         """Sequence index = row (append and per-trajectory attention)."""
         return self._layout(layer, self.row_table)
+
+
+class _ConvState:
+    """The last taps - 1 inputs of every layer's causal convolution, fp32 [n_layer, n_seq, taps - 1, width].
+
+    A forward over several tokens reads one buffer and writes the other (`source` / `target`, then `flip`), so that no
+    thread overwrites what another still reads; one token at a time is updated in place.
+    """
+
+    def __init__(self, n_layer: int, n_seq: int, taps: int, width: int, device) -> None:
+        self.buffers = torch.zeros((2, n_layer, n_seq, taps - 1, width), dtype=torch.float32, device=device)
+        self.current = 0
+
+    @property
+    def source(self) -> torch.Tensor:
+        return self.buffers[self.current]
+
+    @property
+    def target(self) -> torch.Tensor:
+        return self.buffers[1 - self.current]
+
+    def flip(self) -> None:
+        self.current = 1 - self.current
+
+    def clear(self) -> None:
+        self.buffers.zero_()
+        self.current = 0
+
+
+class LatentCache:
+    """Cache of a sliding-window latent-attention model for requests fed step by step.
+
+    ranks      {layer: columns of a cached latent} for the layers that own a latent; other layers read an owner's
+    keep       tokens before a new one that some layer's window can still reach (the largest window less one), or None
+               when a layer sees everything
+    Latents live in one dense run of slots per sequence.  Only the last `keep` tokens are ever needed: when the run is
+    full they move to its front, and `base` (the position of slot 0) moves with them.  Keys carry no positions, so
+    slots are all that the attention kernels need.
+    """
+
+    def __init__(self, batch_size: int, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int,
+                 dtype: torch.dtype, device) -> None:
+        self.batch_size, self.ranks, self.keep = batch_size, ranks, keep
+        self.dtype, self.device = dtype, device
+        self.latents: dict[int, torch.Tensor] = {}
+        self.capacity = 0
+        self.conv = _ConvState(n_layer, batch_size, taps, width, device)
+        self.pos = 0
+        self.base = 0
+
+    def reset(self) -> None:
+        self.pos = self.base = 0
+        self.conv.clear()
+
+    def get_pos(self) -> int:
+        return self.pos
+
+    @property
+    def slot(self) -> int:
+        """The slot the next token goes to."""
+        return self.pos - self.base
+
+    def ensure(self, T: int) -> None:
+        """Make room for T more tokens behind the ones that can still be seen."""
+        if self.slot + T <= self.capacity:
+            return
+        live = self.slot if self.keep is None else min(self.slot, self.keep)
+        first = self.slot - live
+        if live + T <= self.capacity:
+            for t in self.latents.values():
+                t[:, :live] = t[:, first : first + live].clone()
+        else:
+            # room to slide in: as many slots again as stay live (at least 1024), so a move is paid for by many tokens
+            want = (live + T + max(live, 1024) + 63) // 64 * 64
+            for layer, r in self.ranks.items():
+                grown = torch.empty((self.batch_size, want, r), dtype=self.dtype, device=self.device)
+                if live:
+                    grown[:, :live] = self.latents[layer][:, first : first + live]
+                self.latents[layer] = grown
+            self.capacity = want
+        self.base += first
+
+    def layout(self, layer: int) -> ops.KvLayout:
+        c = self.latents[layer]
+        return ops.kv_layout(c, c, page_stride=c.stride(0), head_stride=0, page_tokens=self.capacity)
+
+    def span(self, layer: int, first: int, end: int) -> torch.Tensor:
+        """Latents of slots [first, end) of all sequences as [batch * (end - first), r] (a copy if there are several)."""
+        c = self.latents[layer][:, first:end]
+        return c.reshape(-1, c.shape[-1])
+
+
+class PagedLatentCache:
+    """`PagedKVCache` for latent attention: per owning layer one pool of pages (n_pages, page_tokens, r).
+
+    The prompt's pages are shared by a series' rows.  A row's own pages are a ring when every layer has a window: the
+    table of a row maps each page of generated tokens to physical page (index mod ring length), and the ring is long
+    enough that the page being written is out of every window.  The convolutions' states are kept per series at the
+    prompt's end (`prompts`) and per row (`rows`).
+    """
+
+    prompts_exchangeable = False
+
+    def __init__(self, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int, n_series: int,
+                 rows_per_series: int, prefix_len: int, max_new: int, dtype: torch.dtype, device, page_tokens: int = 64) -> None:
+        pt = self.page_tokens = page_tokens
+        self.n_series, self.rows_per_series = n_series, rows_per_series
+        self.n_rows = n_series * rows_per_series
+        self.prefix_len, self.max_new = prefix_len, max_new
+        self.prefix_pages = max(1, -(-prefix_len // pt))
+        self.own_pages = max(1, -(-max_new // pt))
+        self.ring_pages = self.own_pages if keep is None else min(self.own_pages, -(-keep // pt) + 1)
+        n_pages = n_series * self.prefix_pages + self.n_rows * self.ring_pages
+        self.pools = {layer: torch.zeros((n_pages, pt, r), dtype=dtype, device=device) for layer, r in ranks.items()}
+        pre = torch.arange(n_series * self.prefix_pages, dtype=torch.int32).view(n_series, self.prefix_pages)
+        ring = torch.arange(self.n_rows * self.ring_pages, dtype=torch.int32).view(self.n_rows, self.ring_pages)
+        own = n_series * self.prefix_pages + ring[:, torch.arange(self.own_pages) % self.ring_pages]
+        row = torch.cat([pre.repeat_interleave(rows_per_series, dim=0), own], dim=1)
+        self.prefix_table = pre.contiguous().to(device)
+        self.row_table = row.contiguous().to(device)
+        self.suffix_slot0 = self.prefix_pages * pt
+        self.rows = torch.zeros((n_layer, self.n_rows, taps - 1, width), dtype=torch.float32, device=device)
+        self.prompts: list[tuple[torch.Tensor, torch.Tensor]] = []  # (series indices, their states at the prompt's end)
+
+    @property
+    def bytes(self) -> int:
+        return sum(p.numel() * p.element_size() for p in self.pools.values())
+
+    def prompt_states(self, members: list[int]) -> torch.Tensor:
+        """The convolutions' states of the prompts of these series, [n_layer, len(members), taps - 1, width]."""
+        L, _, k, C = self.rows.shape
+        states = torch.zeros((L, len(members), k, C), dtype=torch.float32, device=self.rows.device)
+        self.prompts.append((torch.tensor(members, device=self.rows.device), states))
+        return states
+
+    def begin_prompts(self) -> None:
+        for _, states in self.prompts:
+            states.zero_()
+
+    def prompts_ready(self) -> None:
+        """Every row starts from the state its series' prompt has left."""
+        L, _, k, C = self.rows.shape
+        rows = self.rows.view(L, self.n_series, self.rows_per_series, k, C)
+        for members, states in self.prompts:
+            rows[:, members] = states.unsqueeze(2).expand(-1, -1, self.rows_per_series, -1, -1)
+
+    def layout(self, layer: int, table: torch.Tensor) -> ops.KvLayout:
+        p = self.pools[layer]
+        return ops.kv_layout(p, p, page_stride=p.stride(0), head_stride=0, page_tokens=self.page_tokens, page_table=table,
+                             n_pages=p.shape[0])

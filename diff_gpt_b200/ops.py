@@ -267,25 +267,27 @@ def linear(
     *,
     swiglu: tuple[float, float] | None = None,
     add: torch.Tensor | None = None,
+    xielu: tuple[float, float] | None = None,
     status: torch.Tensor | None = None,
 ) -> None:
     """out = a @ w.T on the tcgen05 kernel (bf16).  swiglu=(alpha, limit): the SwiGLU of interleaved column pairs is
     applied in the epilogue and `out` has half as many columns as `w` has rows.  add=r: out = r + a @ w.T, rounded
-    once (r may be `out`)."""
+    once (r may be `out`).  xielu=(alpha_p, alpha_n): that activation is applied in the epilogue."""
     _cuda(a, w, out, add, status)
-    assert not (swiglu and add is not None)
+    assert (swiglu is not None) + (add is not None) + (xielu is not None) <= 1
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and a.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
     assert out.shape == (M, N // 2 if swiglu else N) and a.dtype == w.dtype == out.dtype
     if add is not None:
         assert add.shape == out.shape and add.dtype == out.dtype and add.stride(1) == 1
-    alpha, limit = swiglu if swiglu else (0.0, 0.0)
+    alpha, limit = swiglu or xielu or (0.0, 0.0)
+    epilogue = 1 if swiglu else 4 if xielu else 2 if add is not None else 0
     check(
         lib.dgpt_linear(
             a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _ptr(add),
-            0 if add is None else add.stride(0), M, N, K, 1 if swiglu else (2 if add is not None else 0), alpha, limit,
-            dtype_code(a), _ptr(status), _stream(),
+            0 if add is None else add.stride(0), M, N, K, epilogue, alpha, limit, dtype_code(a), _ptr(status),
+            _stream(),
         )
     )
 
@@ -517,3 +519,216 @@ def lmhead_sample(
             _ptr(status), _stream(),
         )
     )
+
+
+# ---- sliding-window / latent attention, fp32 residual stream averaged over depth --------------------
+def fmha_window(
+    q: torch.Tensor,
+    k: torch.Tensor,
+    v: torch.Tensor,
+    o: torch.Tensor,
+    *,
+    B: int,
+    H: int,
+    D: int,
+    n_keys: int,
+    q_offset: int,
+    window: int,
+    scale: float,
+    gate: torch.Tensor | None = None,
+    impl: int = 0,
+    status: torch.Tensor | None = None,
+) -> None:
+    """q, o: [B * Tq, H * D]; k, v: [B * n_keys, H * D]; gate: [B * Tq, H] (2-D views with unit inner stride).
+    Query i of a sequence sees keys (q_offset + i - window, q_offset + i]; window 0 = no lower bound."""
+    _cuda(q, k, v, o, gate, status)
+    n = q.shape[0]
+    assert n % B == 0 and k.shape == v.shape == (B * n_keys, H * D) and q.shape == o.shape == (n, H * D)
+    assert k.stride() == v.stride() and q.stride(1) == k.stride(1) == o.stride(1) == 1
+    assert q.dtype == k.dtype == v.dtype == o.dtype and (gate is None or (gate.shape == (n, H) and gate.stride(1) == 1))
+    Tq = n // B
+    check(
+        lib.dgpt_fmha_window(
+            q.data_ptr(), Tq * q.stride(0), q.stride(0), k.data_ptr(), v.data_ptr(), n_keys * k.stride(0), k.stride(0), D, n_keys,
+            o.data_ptr(), Tq * o.stride(0), o.stride(0), _ptr(gate), 0 if gate is None else gate.stride(0), B, H, Tq, D, q_offset,
+            window, scale, dtype_code(q), impl, _ptr(status), _stream(),
+        )
+    )
+
+
+def latent_append(
+    x: torch.Tensor,
+    w: torch.Tensor,
+    eps: float,
+    kv: KvLayout,
+    slot0: torch.Tensor,
+    step: torch.Tensor | None,
+    *,
+    n_seq: int,
+    T: int,
+    r: int,
+    flat: torch.Tensor | None = None,
+    status: torch.Tensor | None = None,
+) -> None:
+    """x: [n_seq * T, >= w.numel()]; w: fp32 [r_norm]; r: columns of a cached latent (the rest is zero)."""
+    _cuda(x, w, slot0, step, flat, status)
+    assert w.dtype == torch.float32 and slot0.dtype == torch.int32 and x.stride(1) == 1 and x.shape[0] == n_seq * T
+    assert flat is None or (flat.is_contiguous() and flat.dtype == x.dtype and flat.numel() == n_seq * T * r)
+    check(
+        lib.dgpt_latent_append(
+            x.data_ptr(), x.stride(0), w.data_ptr(), eps, w.numel(), C.byref(kv), slot0.data_ptr(), _ptr(step), n_seq, T, r,
+            _ptr(flat), dtype_code(x), _ptr(status), _stream(),
+        )
+    )
+
+
+def latent_attn_workspace_bytes(R: int, H: int, r: int, n_splits: int) -> int:
+    return int(lib.dgpt_latent_attn_workspace_bytes(R, H, r, n_splits))
+
+
+def latent_attn(
+    q: torch.Tensor,
+    kv: KvLayout,
+    len0: torch.Tensor | None,
+    start1: torch.Tensor,
+    len1: torch.Tensor,
+    step: torch.Tensor | None,
+    out: torch.Tensor,
+    *,
+    n_seq: int,
+    T: int,
+    H: int,
+    r: int,
+    window: int,
+    scale: float,
+    gate: torch.Tensor | None = None,
+    workspace: torch.Tensor | None = None,
+    n_splits: int = 1,
+    impl: int = 0,
+) -> None:
+    """q, out: [n_seq * T, H * r]; gate: [n_seq * T, H]."""
+    _cuda(q, len0, start1, len1, step, out, gate, workspace)
+    assert q.shape == out.shape == (n_seq * T, H * r) and q.stride(1) == out.stride(1) == 1 and q.dtype == out.dtype
+    assert gate is None or (gate.shape == (n_seq * T, H) and gate.stride(1) == 1 and gate.dtype == q.dtype)
+    ws_bytes = 0 if workspace is None else workspace.numel() * workspace.element_size()
+    check(
+        lib.dgpt_latent_attn(
+            q.data_ptr(), q.stride(0), C.byref(kv), _ptr(len0), start1.data_ptr(), len1.data_ptr(), _ptr(step), _ptr(gate),
+            0 if gate is None else gate.stride(0), out.data_ptr(), out.stride(0), _ptr(workspace), ws_bytes, n_splits, n_seq, T, H,
+            r, window, scale, dtype_code(q), impl, _stream(),
+        )
+    )
+
+
+def embed_scale(ids: torch.Tensor, emb: torch.Tensor, out: torch.Tensor, scale: float) -> None:
+    _cuda(ids, emb, out)
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and emb.is_contiguous() and out.is_contiguous()
+    assert out.dtype == torch.float32 and out.shape == (ids.numel(), emb.shape[1])
+    V, Cdim = emb.shape
+    check(lib.dgpt_embed_scale(ids.data_ptr(), emb.data_ptr(), out.data_ptr(), ids.numel(), Cdim, V, scale, dtype_code(emb), _stream()))
+
+
+def norm_add(
+    y: torch.Tensor, w: torch.Tensor, eps: float, x: torch.Tensor, out: torch.Tensor, rounded: torch.Tensor | None = None
+) -> None:
+    """out = x + rms_norm(y) * w in fp32; `rounded` receives a copy in y's dtype."""
+    _cuda(y, w, x, out, rounded)
+    for t in (y, w, x, out, rounded):
+        assert t is None or t.is_contiguous()
+    assert w.dtype == x.dtype == out.dtype == torch.float32 and x.shape == out.shape == y.shape
+    assert rounded is None or (rounded.shape == y.shape and rounded.dtype == y.dtype)
+    rows, Cdim = y.shape
+    check(lib.dgpt_norm_add(y.data_ptr(), w.data_ptr(), eps, x.data_ptr(), out.data_ptr(), _ptr(rounded), rows, Cdim, dtype_code(y), _stream()))
+
+
+def _slab(slab: torch.Tensor, terms: int, coef: torch.Tensor) -> None:
+    assert slab.dtype == coef.dtype == torch.float32 and slab.is_contiguous() and slab.dim() == 3
+    assert 1 <= terms <= slab.shape[0] and coef.numel() >= terms and coef.is_contiguous()
+
+
+def depth_avg_conv(
+    slab: torch.Tensor,
+    terms: int,
+    coef: torch.Tensor,
+    conv_w: torch.Tensor,
+    h: torch.Tensor,
+    *,
+    n_seq: int,
+    T: int,
+    x: torch.Tensor | None = None,
+    state_in: torch.Tensor | None = None,
+    state_out: torch.Tensor | None = None,
+) -> None:
+    """slab: fp32 [>= terms, n, C]; conv_w: fp32 [taps, C]; x, h: [n, C]; states: fp32 [n_seq, taps - 1, C]."""
+    _cuda(slab, coef, conv_w, h, x, state_in, state_out)
+    _slab(slab, terms, coef)
+    taps, Cdim = conv_w.shape
+    assert slab.shape[1:] == (n_seq * T, Cdim) and h.shape == (n_seq * T, Cdim) and h.is_contiguous() and conv_w.is_contiguous()
+    assert conv_w.dtype == torch.float32
+    for t in (x, state_in, state_out):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous())
+    for t in (state_in, state_out):
+        assert t is None or t.numel() == n_seq * (taps - 1) * Cdim
+    if taps == 1:
+        state_in = state_out = None
+    check(
+        lib.dgpt_depth_avg_conv(
+            slab.data_ptr(), slab.stride(0), terms, coef.data_ptr(), conv_w.data_ptr(), taps, _ptr(state_in), _ptr(state_out),
+            _ptr(x), h.data_ptr(), n_seq, T, Cdim, dtype_code(h), _stream(),
+        )
+    )
+
+
+def layer_tail(
+    y: torch.Tensor,
+    norm_w: torch.Tensor,
+    eps: float,
+    x1: torch.Tensor,
+    slab: torch.Tensor,
+    terms: int,
+    coef: torch.Tensor,
+    conv_w: torch.Tensor,
+    state: torch.Tensor,
+    x: torch.Tensor,
+    h: torch.Tensor,
+) -> None:
+    """`norm_add` into slab[terms - 1] and `depth_avg_conv` with T = 1 in one launch (one row per sequence)."""
+    _cuda(y, norm_w, x1, slab, coef, conv_w, state, x, h)
+    _slab(slab, terms, coef)
+    taps, Cdim = conv_w.shape
+    rows = y.shape[0]
+    assert x1.data_ptr() != x.data_ptr() and slab.shape[1:] == (rows, Cdim) and conv_w.is_contiguous()
+    for t in (y, x1, x, h):
+        assert t.shape == (rows, Cdim) and t.is_contiguous()
+    assert x1.dtype == x.dtype == norm_w.dtype == conv_w.dtype == torch.float32 and y.dtype == h.dtype
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.numel() == rows * (taps - 1) * Cdim
+    check(
+        lib.dgpt_layer_tail(
+            y.data_ptr(), norm_w.data_ptr(), eps, x1.data_ptr(), slab.data_ptr(), slab.stride(0), terms, coef.data_ptr(),
+            conv_w.data_ptr(), taps, state.data_ptr() if taps > 1 else None, x.data_ptr(), h.data_ptr(), rows, Cdim, dtype_code(y),
+            _stream(),
+        )
+    )
+
+
+def depth_avg_norm(
+    slab: torch.Tensor, terms: int, coef: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None
+) -> None:
+    """out = rms_norm(sum_j coef[j] slab[j]) * w for the rows named by `rows` (int32, None = the first out.shape[0])."""
+    _cuda(slab, coef, w, out, rows)
+    _slab(slab, terms, coef)
+    n, Cdim = slab.shape[1:]
+    assert w.dtype == torch.float32 and w.numel() == Cdim and out.is_contiguous() and out.shape[1] == Cdim
+    assert rows is None or (rows.dtype == torch.int32 and rows.is_contiguous() and rows.numel() == out.shape[0])
+    check(
+        lib.dgpt_depth_avg_norm(
+            slab.data_ptr(), slab.stride(0), terms, coef.data_ptr(), w.data_ptr(), eps, _ptr(rows), out.data_ptr(), out.shape[0],
+            n, Cdim, dtype_code(out), _stream(),
+        )
+    )
+
+
+def xielu(x: torch.Tensor, out: torch.Tensor, alpha_p: float, alpha_n: float) -> None:
+    _cuda(x, out)
+    assert x.is_contiguous() and out.is_contiguous() and x.shape == out.shape and x.dtype == out.dtype
+    check(lib.dgpt_xielu(x.data_ptr(), out.data_ptr(), x.numel(), alpha_p, alpha_n, dtype_code(x), _stream()))

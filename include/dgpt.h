@@ -215,9 +215,10 @@ int dgpt_softcap(void* logits, int64_t n, float cap, int32_t dtype, void* stream
  *   epilogue 1:  out[m, n / 2] = swiglu(acc[m, n], acc[m, n + 1]) for even n, the rule of dgpt_swiglu applied to
  *                the accumulator rounded to bf16 (as the reference's Linear output is)      out: [M, N / 2]
  *   epilogue 2:  out[m, n]     = resid[m, n] + acc[m, n], rounded once (resid may be out itself)   out: [M, N]
+ *   epilogue 4:  out[m, n]     = xielu(acc[m, n]) with alpha_p = alpha, alpha_n = limit (see dgpt_xielu)   out: [M, N]
  * Replaces nn.Linear of src/diff_gpt/model/feed_forward.py:10-14 followed by swi_glu.py:11-19 (epilogue 1), any
  * bias-free nn.Linear of the path (epilogue 0), or a projection with the residual add that follows it
- * (src/diff_gpt/model/block.py:98-106, epilogue 2).  resid is ignored for epilogues 0 and 1.  bf16 only; pointers 16-byte aligned, K and the row strides
+ * (src/diff_gpt/model/block.py:98-106, epilogue 2).  resid is ignored for epilogues 0, 1 and 4.  bf16 only; pointers 16-byte aligned, K and the row strides
  * multiples of 8 elements, N a multiple of 16.  status: device int32, set non-zero if a bounded wait ran out. */
 int dgpt_linear(const void* a, int64_t a_row_stride, const void* w, int64_t w_row_stride, void* out,
                 int64_t out_row_stride, const void* resid, int64_t resid_row_stride, int32_t M, int32_t N,
@@ -334,6 +335,78 @@ int dgpt_lmhead_sample(const void* xn, int64_t xn_row_stride, const void* emb, i
 int dgpt_nucleus_filter(const void* logits, int64_t logits_row_stride, void* filtered,
                         int64_t filtered_row_stride, int32_t R, int32_t V, float top_p, int32_t dtype,
                         void* stream);
+
+/* ---- sliding-window and latent attention; models with an fp32 residual stream averaged over depth ----------------
+ * (No counterpart in the reference project: these serve model designs beyond its GPT.) */
+
+/* Sliding-window attention with expanded keys and values:
+ *   o[b,i,h,:] = sigmoid(gate[b,i,h]) * sum_j p_j v[b,j,h,:],  p = softmax_j(q[b,i,h,:] . k[b,j,h,:] * scale)
+ * over keys j < n_keys with q_offset + i - window < j <= q_offset + i (window 0: every j <= q_offset + i).
+ * q: element (b,i,h,d) at b*q_batch_stride + i*q_row_stride + h*D + d; o likewise; k, v: element (b,j,h,d) at
+ * b*kv_batch_stride + j*kv_row_stride + h*kv_head_stride + d (strides in elements, multiples of 8; pointers 16-byte
+ * aligned).  gate: [B * Tq, H] in dtype with gate_row_stride, or NULL.
+ * The kernels are those of dgpt_fmha_prefill (bf16 with D = 32, 64, 128 on the tcgen05 tensor cores, else the warp-level
+ * kernel with D in {8, 16, 32, 64, 128}); key tiles that lie outside every window of a query tile are not visited.
+ * impl: 0 = choose, 1 = warp-level, 2 = persistent tensor-core kernel, 3 = the small tensor-core kernel. */
+int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const void* k, const void* v,
+                     int64_t kv_batch_stride, int64_t kv_row_stride, int64_t kv_head_stride, int32_t n_keys, void* o,
+                     int64_t o_batch_stride, int64_t o_row_stride, const void* gate, int64_t gate_row_stride, int32_t B,
+                     int32_t H, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, float scale, int32_t dtype,
+                     int32_t impl, int32_t* status, void* stream);
+
+/* c = x / sqrt(mean(x[0..r_norm)^2) + eps) * w, rounded once and appended to a latent cache.  Token (s, t) goes to slot
+ * seq_slot0[s] + step + t of sequence s; latent `slot` of a sequence lives at page * page_stride + (slot % page_tokens) * r
+ * from kv->k_base (kv->v_base must name the same storage; head_stride is not used).  Columns r_norm..r-1 are written as
+ * zeros.  in: device [n_seq*T] rows of >= r_norm numbers; w: device fp32 [r_norm]; r: a multiple of 8;
+ * flat: device [n_seq*T, r] or NULL, receives the same rows contiguously; status: as in dgpt_rope_qknorm_kvappend. */
+int dgpt_latent_append(const void* in, int64_t in_row_stride, const float* w, float eps, int32_t r_norm,
+                       const dgpt_kv_layout* kv, const int32_t* seq_slot0, const int32_t* step_ptr, int32_t n_seq, int32_t T,
+                       int32_t r, void* flat, int32_t dtype, int32_t* status, void* stream);
+
+/* Attention on cached latents, shared by all heads, key and value expansions absorbed into q and the output projection:
+ *   out[row,h,:] = sigmoid(gate[row,h]) * sum_j p_j c_j,   p = softmax_j(q[row,h,:] . c_j * scale)
+ * row = s * T + t.  Row (s, t) sees the last `window` (0 = all) of the keys 0 .. n-1, n = len0[s] + len1[s] + step + t,
+ * where key i is slot i for i < len0[s] and slot start1[s] + i - len0[s] from there on (len0 NULL = 0).
+ * q, out: device [n_seq*T, H*r] with row strides; gate: [n_seq*T, H] in dtype or NULL; r a multiple of 8.
+ * n_splits > 1 splits each row's keys over CTAs (workspace from the _bytes call with R = n_seq * T, 16-byte aligned).
+ * impl: 0 = choose, 1 = CUDA cores (any r), 2 = tensor cores (bf16, r <= 512) or fail. */
+size_t dgpt_latent_attn_workspace_bytes(int32_t R, int32_t H, int32_t r, int32_t n_splits);
+int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, const int32_t* len0, const int32_t* start1,
+                     const int32_t* len1, const int32_t* step_ptr, const void* gate, int64_t gate_row_stride, void* out,
+                     int64_t out_row_stride, void* workspace, size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T,
+                     int32_t H, int32_t r, int32_t window, float scale, int32_t dtype, int32_t impl, void* stream);
+
+/* out = scale * emb[ids] in fp32.  ids: device int32 [n_tokens]; emb: [V, C] in dtype; out: fp32 [n_tokens, C]. */
+int dgpt_embed_scale(const int32_t* ids, const void* emb, float* out, int64_t n_tokens, int32_t C, int32_t V, float scale,
+                     int32_t dtype, void* stream);
+
+/* out = x + y / sqrt(mean(y^2) + eps) * w: the norm on a sublayer's output and the residual sum, in fp32.
+ * y: [rows, C] in dtype; w: fp32 [C]; x, out: fp32 [rows, C] (may alias); u: [rows, C] in dtype or NULL, a rounded copy. */
+int dgpt_norm_add(const void* y, const float* w, float eps, const float* x, float* out, void* u, int64_t rows, int32_t C,
+                  int32_t dtype, void* stream);
+
+/* Weighted average over depth and the causal convolution in front of the next mixer:
+ *   x[s,t] = sum_{j < terms} coef[j] * slab[j][s,t],    h[s,t] = x[s,t] + sum_{k < taps} conv_w[k] * x[s, t - taps + 1 + k]
+ * per channel.  slab: fp32, term j at j * term_stride, rows s * T + t; coef: device fp32 [terms]; conv_w: device fp32
+ * [taps, C] (tap-major); state_in: fp32 [n_seq, taps - 1, C], the last taps - 1 x of each sequence before the call, or NULL
+ * (zeros); state_out: the same after the call, or NULL (may be state_in only for T = 1); x_out: fp32 or NULL; h_out: dtype.
+ * taps <= 16. */
+int dgpt_depth_avg_conv(const float* slab, int64_t term_stride, int32_t terms, const float* coef, const float* conv_w,
+                        int32_t taps, const float* state_in, float* state_out, float* x_out, void* h_out, int32_t n_seq,
+                        int32_t T, int32_t C, int32_t dtype, void* stream);
+
+/* One new token per sequence: dgpt_norm_add into slab term terms - 1, then dgpt_depth_avg_conv with T = 1 on the `terms`
+ * terms, state [rows, taps - 1, C] updated in place.  x1 must not be x_out. */
+int dgpt_layer_tail(const void* y, const float* norm_w, float eps, const float* x1, float* slab, int64_t term_stride,
+                    int32_t terms, const float* coef, const float* conv_w, int32_t taps, float* state, float* x_out,
+                    void* h_out, int64_t rows, int32_t C, int32_t dtype, void* stream);
+
+/* out[i] = rms_norm(sum_j coef[j] slab[j][row_index[i]]) * w in dtype (row_index NULL = the first n_out of the n rows). */
+int dgpt_depth_avg_norm(const float* slab, int64_t term_stride, int32_t terms, const float* coef, const float* w, float eps,
+                        const int32_t* row_index, void* out, int64_t n_out, int64_t n, int32_t C, int32_t dtype, void* stream);
+
+/* out[i] = alpha_p z^2 + z / 2 for z = in[i] > 0,  alpha_n (e^z - 1 - z) + z / 2 otherwise.  in, out: device [n] in dtype. */
+int dgpt_xielu(const void* in, void* out, int64_t n, float alpha_p, float alpha_n, int32_t dtype, void* stream);
 
 #ifdef __cplusplus
 }
