@@ -1056,6 +1056,244 @@ def kernel_case(name: str, iters: int = 8) -> None:
                       "frac": rate / peak, "algorithmic_work_per_launch": work, "peak_source": pk["source"]}), flush=True)
 
 
+# ---------------------------------------------------------------------------------------
+# The Delunex design beside this package's GPT at equal size (--design delunex)
+# ---------------------------------------------------------------------------------------
+# layers of a real model's shape, a few of them; every other layer reads the latent of the one before
+DESIGN_SIZES = {
+    "w1024": dict(width=1024, heads=16, dim=64, kv_rank=256, ff=4096, window=512, layers=8, vocab=16384),
+    "w2048": dict(width=2048, heads=16, dim=128, kv_rank=512, ff=8192, window=1024, layers=8, vocab=16384),
+    "w2048_long": dict(width=2048, heads=16, dim=128, kv_rank=256, ff=8192, window=4096, layers=8, vocab=16384),
+}
+
+
+def design_config(z: dict) -> dict:
+    layers = []
+    for i in range(z["layers"]):
+        m = dict(heads=z["heads"], dim=z["dim"], vdim=z["dim"], kv_rank=z["kv_rank"], scale=z["dim"] ** -0.5, mask={"size": z["window"]})
+        if i % 2:
+            m["kv_from"] = i - 1
+        layers.append({"type": "latent_attention", "mixer": m, "mlp": {"kind": "dense", "ff": z["ff"]}})
+    return {"architecture": "Delunex", "width": z["width"], "vocab": z["vocab"], "canon": {"taps": 4}, "norm": {"eps": 1e-6},
+            "embedding": {"scale": z["width"] ** 0.5}, "logit_scale": 1.0, "layers": layers}
+
+
+def design_model(kind: str, z: dict, dev):
+    """Random-weight model of the design or this package's GPT at the same width, heads, depth and vocabulary."""
+    from diff_gpt_b200 import Delunex, GPT
+
+    g = torch.Generator(device=dev).manual_seed(1)
+    with torch.device(dev):
+        if kind == "delunex":
+            m = Delunex(design_config(z))
+        else:
+            m = GPT(vocab_size=z["vocab"], n_embd=z["width"], n_head=z["heads"], n_layer=z["layers"], block_size=16384)
+    m = m.to(torch.bfloat16).to(dev).eval()
+    with torch.no_grad():
+        for p in m.parameters():
+            p.copy_(torch.randn(p.shape, device=dev, generator=g) * 0.02)
+    return m
+
+
+def event_ms(fn, iters: int, warm: int = 3) -> float:
+    for _ in range(warm):
+        fn()
+    torch.cuda.synchronize()
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(iters):
+        fn()
+    b.record()
+    torch.cuda.synchronize()
+    return a.elapsed_time(b) / iters
+
+
+def graph_ms(launch, iters: int) -> float:
+    """Device time per launch, replayed from a CUDA graph (a Python call costs more than some kernels run)."""
+    for _ in range(3):
+        launch()
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for _ in range(iters):
+            launch()
+    graph.replay()
+    torch.cuda.synchronize()
+    return event_ms(graph.replay, 3, 1) / iters
+
+
+def design_throughput(kind: str, z: dict, dev, rows: int, prompt: int, steps: int, prefill: tuple) -> dict:
+    """Prefill (one plan, last-position logits) and decode (captured step, `rows` requests of `prompt` tokens each)."""
+    from diff_gpt_b200 import TemperatureSampler, _lib
+    from diff_gpt_b200.model.engine import DecodeRun
+
+    m = design_model(kind, z, dev)
+    g = torch.Generator(device=dev).manual_seed(2)
+    out = {}
+    with torch.inference_mode():
+        for B, T in prefill:
+            cache = m.paged_cache(B, 1, T, 1, 64)
+            bind, plan = m.prefill_plan(cache, list(range(B)), T, 0)
+            ids = torch.randint(0, z["vocab"], (B * T,), device=dev, generator=g, dtype=torch.int32)
+            ms = event_ms(lambda: plan.run(ids, bind), 5)
+            assert int(plan.status.item()) == 0
+            out[f"prefill_{B}x{T}"] = {"ms": ms, "tokens_per_s": B * T / ms * 1e3}
+            timer = _lib.KernelTimer()
+            with _lib.timed(timer):
+                plan.run(ids, bind)
+            torch.cuda.synchronize()
+            out[f"prefill_{B}x{T}"]["kernels_us"] = {k: [v["launches"], round(1e3 * v["total_ms"], 1)] for k, v in timer.summary().items()}
+            del cache, bind, plan
+        for R in (1, rows):
+            ids = torch.randint(0, z["vocab"], (R, prompt), device=dev, generator=g, dtype=torch.int32)
+            run = DecodeRun(m, ids, 1, steps + 8, TemperatureSampler(1.0), 42, None)
+            run.start()
+            run.advance(5)
+            torch.cuda.synchronize()
+            ms = event_ms(lambda: run.advance(1), steps, 0)
+            run.check_status()
+            out[f"decode_{R}rows"] = {"ms_per_step": ms, "tokens_per_s": R / ms * 1e3, "prompt": prompt}
+            del run
+            torch.cuda.empty_cache()
+    return out
+
+
+def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
+    """Each hot kernel of the design alone, then the like kernel of the GPT, at one size: time, rate and fraction of the
+    measured peak.  Inputs larger than the L2, or several sets of them in turn."""
+    from diff_gpt_b200 import ops
+
+    pk = peaks()
+    g = torch.Generator(device=dev).manual_seed(0)
+    bf, f32 = torch.bfloat16, torch.float32
+    C, H, D, r, W, ff = z["width"], z["heads"], z["dim"], z["kv_rank"], z["window"], z["ff"]
+
+    def rnd(*s, dtype=bf):
+        return torch.randn(s, device=dev, generator=g, dtype=f32).to(dtype)
+
+    out = {}
+
+    def report(name, launch, iters, nbytes=None, flops=None):
+        ms = graph_ms(launch, iters)
+        if flops is not None and (nbytes is None or flops / (pk["bf16_tflops"] * 1e12) > nbytes / (pk["hbm_gbs"] * 1e9)):
+            rate, peak, unit = flops / ms / 1e9, pk["bf16_tflops"], "TFLOP/s"
+        else:
+            rate, peak, unit = nbytes / ms / 1e6, pk["hbm_gbs"], "GB/s"
+        out[name] = {"us": 1e3 * ms, "rate": rate, "unit": unit, "frac": rate / peak}
+
+    def in_turn(sets, fn):
+        turn = [0]
+
+        def launch():
+            fn(*sets[turn[0] % len(sets)])
+            turn[0] += 1
+
+        return launch
+
+    def copies(nbytes):  # sets of inputs that together are well beyond the 126 MB L2
+        return max(1, min(16, -(-400_000_000 // nbytes)))
+
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    # ---- decode attention over latents: rows x W keys ----
+    pt, per = 64, -(-W // 64)
+    pool = rnd(rows * per, pt, r)
+    table = torch.randperm(rows * per, device=dev, generator=g).to(torch.int32).view(rows, per)
+    lay = ops.kv_layout(pool, pool, pt * r, 0, pt, table, n_pages=rows * per)
+    q, gate, o = rnd(rows, H * r), rnd(rows, H), torch.empty((rows, H * r), device=dev, dtype=bf)
+    zero, n1 = torch.zeros(rows, dtype=torch.int32, device=dev), torch.full((rows,), W, dtype=torch.int32, device=dev)
+    from diff_gpt_b200.model.delunex import pick_latent_splits
+
+    splits = pick_latent_splits(rows, -(-H // 64), W)
+    ws = torch.empty(max(4, ops.latent_attn_workspace_bytes(rows, H, r, splits) // 4), device=dev) if splits > 1 else None
+    report("latent_attn", lambda: ops.latent_attn(q, lay, None, zero, n1, None, o, n_seq=rows, T=1, H=H, r=r, window=W, scale=D**-0.5,
+                                                  gate=gate, workspace=ws, n_splits=splits, status=st),
+           8, rows * (W * r + 2 * H * r + H) * 2, 4 * rows * H * W * r)
+    del pool
+    # ---- prefill attention with a window ----
+    proj, kv, o = rnd(T, H * D), rnd(T, 2 * H * D), torch.empty((T, H * D), device=dev, dtype=bf)
+    gate = rnd(T, H)
+    seen = T * W - W * (W - 1) // 2 if T >= W else T * (T + 1) // 2
+    report("fmha_window", lambda: ops.fmha_window(proj, kv[:, : H * D], kv[:, H * D :], o, B=1, H=H, D=D, n_keys=T, q_offset=0, window=W,
+                                                  scale=D**-0.5, gate=gate, status=st), 8, None, 4 * D * H * seen)
+    # ---- element-wise kernels of a prefill ----
+    terms = z["layers"] // 2 + 1
+    slab, a, cw = rnd(terms, T, C, dtype=f32), rnd(terms, dtype=f32), rnd(4, C, dtype=f32)
+    x, h, y, u, w = rnd(T, C, dtype=f32), rnd(T, C), rnd(T, C), rnd(T, C), rnd(C, dtype=f32)
+    report("depth_avg_conv", lambda: ops.depth_avg_conv(slab, terms, a, cw, h, n_seq=1, T=T, x=x), 8, T * C * (4 * terms + 6))
+    sets = [(rnd(T, C), rnd(T, C, dtype=f32), rnd(T, C, dtype=f32), rnd(T, C)) for _ in range(copies(T * C * 12))]
+    report("norm_add", in_turn(sets, lambda yy, xx, oo, uu: ops.norm_add(yy, w, 1e-6, xx, oo, rounded=uu)), 8, T * C * 12)
+    lat, lw = rnd(T, r + 8), rnd(r, dtype=f32)
+    lc = torch.empty((1, T, r), device=dev, dtype=bf)
+    ll = ops.kv_layout(lc, lc, T * r, 0, T)
+    z1 = torch.zeros(1, dtype=torch.int32, device=dev)
+    report("latent_append", lambda: ops.latent_append(lat[:, :r], lw, 1e-6, ll, z1, None, n_seq=1, T=T, r=r, status=st), 8, T * r * 4)
+    # ---- one-pass tail of a decoded layer ----
+    n_set = copies(rows * C * (2 + 4 + 4 * (terms + 1) + 24 + 2))
+    tails = [(rnd(rows, C), rnd(rows, C, dtype=f32), rnd(terms, rows, C, dtype=f32), rnd(rows, 3, C, dtype=f32), rnd(rows, C, dtype=f32), rnd(rows, C))
+             for _ in range(n_set)]
+    report("layer_tail", in_turn(tails, lambda yy, x1, sl, stt, xo, ho: ops.layer_tail(yy, w, 1e-6, x1, sl, terms, a, cw, stt, xo, ho)),
+           16, rows * C * (2 + 4 + 4 * terms + 24 + 4 + 2))
+    del sets, tails, slab
+    # ---- feed-forward GEMM with the activation ----
+    wu, act = rnd(ff, C), torch.empty((T, ff), device=dev, dtype=bf)
+    report("linear_xielu", lambda: ops.linear(u, wu, act, xielu=(0.8, 1.1), status=st), 8, None, 2 * T * ff * C)
+    report("cublas_up", lambda: torch.mm(u, wu.t(), out=act), 8, None, 2 * T * ff * C)
+
+    # ---- the like kernels of the GPT at this size ----
+    Dg = C // H
+    pool = rnd(rows * per, 2, H, pt, Dg)
+    lay = ops.kv_layout(pool[0, 0], pool[0, 1], 2 * H * pt * Dg, pt * Dg, pt, table, n_pages=rows * per)
+    q, gate, o = rnd(rows, C), rnd(rows, C), torch.empty((rows, C), device=dev, dtype=bf)
+    report("gpt.decode_attn", lambda: ops.decode_attn(q, lay, zero, zero, n1, None, o, H=H, D=Dg, gate=gate), 8,
+           rows * (2 * C * W + 3 * C) * 2)
+    del pool
+    q = rnd(T, C)
+    kv = rnd(2, H, T, Dg)
+    lay = ops.kv_layout(kv[0], kv[1], 2 * H * T * Dg, T * Dg, T)
+    o = torch.empty_like(q)
+    report("gpt.fmha_prefill", lambda: ops.fmha_prefill(q, lay, o, B=1, H=H, Tq=T, D=Dg, q_batch_stride=T * C, q_row_stride=C,
+                                                        o_batch_stride=T * C, o_row_stride=C, kv_len_all=T, causal=True, status=st),
+           8, None, 4 * Dg * H * (T * (T + 1) // 2))
+    cands = [rnd(T, C) for _ in range(terms)]
+    wq = rnd(C)
+    report("gpt.depthmix", lambda: ops.depthmix(cands, wq, None, u), 8, T * C * 2 * (terms + 1))
+    small = [([rnd(rows, C) for _ in range(terms)], rnd(rows, C)) for _ in range(copies(rows * C * 2 * (terms + 1)))]
+    report("gpt.depthmix_decode", in_turn(small, lambda cc, oo: ops.depthmix(cc, wq, None, oo)), 16, rows * C * 2 * (terms + 1))
+    act2 = torch.empty((T, ff // 2), device=dev, dtype=bf)
+    report("gpt.linear_swiglu", lambda: ops.linear(u, wu, act2, swiglu=(1.702, 7.0), status=st), 8, None, 2 * T * ff * C)
+    qkvg = rnd(T, 4 * C)
+    qo = torch.empty((T, C), device=dev, dtype=bf)
+    tab = rnd(T, Dg // 2, 2)
+    report("gpt.rope_append", lambda: ops.rope_qknorm_kvappend(qkvg[:, :C], qkvg[:, C : 2 * C], qkvg[:, 2 * C : 3 * C], qo, tab, lay, z1, z1,
+                                                               None, 1, T, H, Dg, st), 8, T * C * 2 * 6)
+    gate = rnd(T, C)
+    report("gpt.sigmoid_gate", lambda: ops.sigmoid_gate(qo, gate), 8, T * C * 2 * 3)
+    assert int(st.item()) == 0
+    return out
+
+
+def run_design(args) -> None:
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    clocks = ClockSampler(0)
+    line = {"design": args.design, "dtype": "bf16", "data": "synthetic tokens, random weights", "sizes": {}}
+    names = args.sizes.split(",") if args.sizes else list(DESIGN_SIZES)
+    for name in names:
+        z = DESIGN_SIZES[name]
+        rows, prompt, T = 256, 2 * z["window"] if z["window"] <= 1024 else z["window"], 8192
+        entry = {"config": z}
+        if not args.kernels_only:
+            for kind in ("delunex", "gpt"):
+                entry[kind] = design_throughput(kind, z, dev, rows, prompt, 32, ((1, T), (8, 2048)))
+                torch.cuda.empty_cache()
+        entry["kernels"] = design_kernels(z, dev, rows, T)
+        torch.cuda.empty_cache()
+        line["sizes"][name] = entry
+    line["clocks"] = clocks.stop()
+    line["peaks"] = peaks()
+    emit(line)
+
+
 def main() -> None:
     ap = argparse.ArgumentParser()
     ap.add_argument("--kernel-case", default=None, choices=["decode_attn", "fmha", "fmha_long", "fmha_pair", "sample", "depthmix", "fmha_prefix", "linear"],
@@ -1075,6 +1313,11 @@ def main() -> None:
     ap.add_argument("--no-graph", action="store_true", help="launch the decode steps eagerly (for profilers)")
     ap.add_argument("--small", action="store_true",
                     help="profiling case: 2048 trajectories x 64 steps (4.8 GB of KV), same model and prompt")
+    ap.add_argument("--design", default=None, choices=["delunex"],
+                    help="instead of the workload above: prefill and decode throughput of this model design beside the GPT at "
+                         "equal size, and its kernels beside the GPT's like ones; one JSON line")
+    ap.add_argument("--sizes", default=None, help="with --design: comma-separated names out of " + ", ".join(DESIGN_SIZES))
+    ap.add_argument("--kernels-only", action="store_true", help="with --design: the kernel table alone")
     args = ap.parse_args()
     if args.small:
         globals().update(TRAJECTORIES=2048, HORIZON=64)
@@ -1082,6 +1325,9 @@ def main() -> None:
         kernel_case(args.kernel_case)
         return
     claim_stdout()
+    if args.design:
+        run_design(args)
+        return
     if args.impl == "reference":
         run_reference(args)
     else:

@@ -11,4 +11,12 @@ __device__ __forceinline__ float xielu_value(float z, float alpha_p, float alpha
   return fmaf(0.5f, z, curve);
 }
 
+// The same for a result that is rounded to bf16: e^z from the exponential unit, with an absolute error near 1e-7 (below
+// a bf16 step of the sum wherever that is larger than 1e-4), a third of the instructions.
+__device__ __forceinline__ float xielu_fast(float z, float alpha_p, float alpha_n) {
+  const bool pos = z > 0.f;
+  const float t = pos ? z * z : __expf(z) - 1.f - z;
+  return fmaf(pos ? alpha_p : alpha_n, t, 0.5f * z);
+}
+
 }  // namespace dgpt

@@ -237,7 +237,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ C
               for (int x = 0; x < 8; ++x) v[8 * q + x] += r8[x];
             } else if (p.mode == 4) {
 #pragma unroll
-              for (int x = 0; x < 8; ++x) v[8 * q + x] = xielu_value(v[8 * q + x], p.alpha, p.limit);
+              for (int x = 0; x < 8; ++x) v[8 * q + x] = xielu_fast(v[8 * q + x], p.alpha, p.limit);
             }
             st16<__nv_bfloat16>(dst + 8 * q, v + 8 * q, 1.f);
           }

@@ -393,9 +393,9 @@ extern "C" int dgpt_depth_avg_conv(const float* slab, int64_t term_stride, int32
   const bool v4 = C % 4 == 0 && term_stride % 4 == 0 && al16(slab) && al16(conv_w) && al16(state_in) && al16(state_out) &&
                   al16(x_out) && al16(h_out);
   const int cv = v4 ? C / 4 : C;
-  // long runs average fewer tokens twice, short ones give more threads: about four waves of 2048 threads per SM
+  // long runs average fewer tokens twice, short ones give more threads: half of what the SMs hold is enough
   int seg = 16;
-  while (seg > 1 && (long long)n_seq * ((T + seg - 1) / seg) * cv < 4ll * 148 * 2048) seg >>= 1;
+  while (seg > 1 && (long long)n_seq * ((T + seg - 1) / seg) * cv < 148ll * 1024) seg >>= 1;
   const int n_seg = (T + seg - 1) / seg;
   const long long work = (long long)n_seq * n_seg * cv;
   const unsigned grid = (unsigned)((work + 127) / 128);

@@ -212,12 +212,11 @@ def _fp32_reductions():
 
 
 def pick_latent_splits(rows: int, head_groups: int, keys: int) -> int:
-    """CTAs per row along the keys: enough to give every multiprocessor two, at least one 64-key tile each."""
+    """CTAs per row along the keys: enough that every multiprocessor has one, each with a 128-key tile at least."""
     ctas = max(1, rows * head_groups)
-    target = 2 * _sm_count()
-    if ctas >= target or keys <= 64:
+    if ctas >= _sm_count() or keys <= 128:
         return 1
-    return max(1, min(-(-target // ctas), -(-keys // 64), 64))
+    return max(1, min(_sm_count() // ctas, -(-keys // 128), 64))
 
 
 class DelunexPlan:
@@ -287,13 +286,13 @@ class DelunexPlan:
             qa, oa = self._buf("qa", n, H * r), self._buf("oa", n, H * r)
             with region("gemm_absorb"):
                 torch.bmm(q.view(n, H, D).transpose(0, 1), lw.w_uk, out=qa.view(n, H, r).transpose(0, 1))
-            splits = pick_latent_splits(n, -(-H // 16), min(b.keys, lw.window))
+            splits = pick_latent_splits(n, -(-H // 64), min(b.keys, lw.window))
             ws = None
             if splits > 1:
                 ws = self._buf("ws", ops.latent_attn_workspace_bytes(n, H, r, splits) // 4, dtype=torch.float32)
             ops.latent_attn(
                 qa, b.layout(lw.owner), b.len0, b.start1, b.len1, b.step, oa, n_seq=n_seq, T=T, H=H, r=r, window=lw.window,
-                scale=lw.scale, gate=gate, workspace=ws, n_splits=splits,
+                scale=lw.scale, gate=gate, workspace=ws, n_splits=splits, status=self.status,
             )
             with region("gemm_absorb"):
                 torch.bmm(oa.view(n, H, r).transpose(0, 1), lw.w_uv_t, out=o.view(n, H, D).transpose(0, 1))

@@ -605,9 +605,10 @@ def latent_attn(
     workspace: torch.Tensor | None = None,
     n_splits: int = 1,
     impl: int = 0,
+    status: torch.Tensor | None = None,
 ) -> None:
     """q, out: [n_seq * T, H * r]; gate: [n_seq * T, H]."""
-    _cuda(q, len0, start1, len1, step, out, gate, workspace)
+    _cuda(q, len0, start1, len1, step, out, gate, workspace, status)
     assert q.shape == out.shape == (n_seq * T, H * r) and q.stride(1) == out.stride(1) == 1 and q.dtype == out.dtype
     assert gate is None or (gate.shape == (n_seq * T, H) and gate.stride(1) == 1 and gate.dtype == q.dtype)
     ws_bytes = 0 if workspace is None else workspace.numel() * workspace.element_size()
@@ -615,7 +616,7 @@ def latent_attn(
         lib.dgpt_latent_attn(
             q.data_ptr(), q.stride(0), C.byref(kv), _ptr(len0), start1.data_ptr(), len1.data_ptr(), _ptr(step), _ptr(gate),
             0 if gate is None else gate.stride(0), out.data_ptr(), out.stride(0), _ptr(workspace), ws_bytes, n_splits, n_seq, T, H,
-            r, window, scale, dtype_code(q), impl, _stream(),
+            r, window, scale, dtype_code(q), impl, _ptr(status), _stream(),
         )
     )
 

@@ -369,12 +369,13 @@ int dgpt_latent_append(const void* in, int64_t in_row_stride, const float* w, fl
  * where key i is slot i for i < len0[s] and slot start1[s] + i - len0[s] from there on (len0 NULL = 0).
  * q, out: device [n_seq*T, H*r] with row strides; gate: [n_seq*T, H] in dtype or NULL; r a multiple of 8.
  * n_splits > 1 splits each row's keys over CTAs (workspace from the _bytes call with R = n_seq * T, 16-byte aligned).
- * impl: 0 = choose, 1 = CUDA cores (any r), 2 = tensor cores (bf16, r <= 512) or fail. */
+ * impl: 0 = choose, 1 = CUDA cores (any r), 2 = tcgen05 (bf16, r <= 512, a dense run of slots per sequence or pages of 8 to
+ * 64 or a multiple of 128 tokens) or fail.  status: device int32, set non-zero if a bounded wait ran out. */
 size_t dgpt_latent_attn_workspace_bytes(int32_t R, int32_t H, int32_t r, int32_t n_splits);
 int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, const int32_t* len0, const int32_t* start1,
                      const int32_t* len1, const int32_t* step_ptr, const void* gate, int64_t gate_row_stride, void* out,
                      int64_t out_row_stride, void* workspace, size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T,
-                     int32_t H, int32_t r, int32_t window, float scale, int32_t dtype, int32_t impl, void* stream);
+                     int32_t H, int32_t r, int32_t window, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream);
 
 /* out = scale * emb[ids] in fp32.  ids: device int32 [n_tokens]; emb: [V, C] in dtype; out: fp32 [n_tokens, C]. */
 int dgpt_embed_scale(const int32_t* ids, const void* emb, float* out, int64_t n_tokens, int32_t C, int32_t V, float scale,

@@ -179,9 +179,9 @@ def test_split_policy():
     from diff_gpt_b200.model.delunex import pick_latent_splits
 
     assert pick_latent_splits(4096, 1, 1024) == 1
-    assert pick_latent_splits(1, 1, 64) == 1
-    assert pick_latent_splits(1, 1, 1024) == 16  # one tile each
-    assert 1 < pick_latent_splits(32, 1, 4096) <= 64
+    assert pick_latent_splits(1, 1, 128) == 1
+    assert pick_latent_splits(1, 1, 1024) == 8  # one tile each
+    assert pick_latent_splits(32, 1, 4096) == 4 and pick_latent_splits(1, 1, 10**6) == 64
 
 
 # ---- the plain implementation: facts that do not depend on the product ------------------------

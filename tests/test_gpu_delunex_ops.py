@@ -204,11 +204,14 @@ def test_latent_attention(dtype, case):
     ws = torch.empty(ops.latent_attn_workspace_bytes(B * T, H, r, splits) // 4, device="cuda") if splits > 1 else None
     start = torch.zeros(B, dtype=torch.int32, device="cuda")
     n1 = torch.tensor(lens, dtype=torch.int32, device="cuda")
-    impls = [0, 1] if dtype == torch.bfloat16 and r <= 512 else [0]
+    impls = [0, 1] if dtype == torch.bfloat16 else [0]
+    status = torch.zeros(1, dtype=torch.int32, device="cuda")
     for impl in impls:
         out.fill_(float("nan"))
         ops.latent_attn(q.reshape(B * T, H * r).cuda(), lay, None, start, n1, None, out, n_seq=B, T=T, H=H, r=r, window=window,
-                        scale=scale, gate=gate.reshape(B * T, H).cuda(), workspace=ws, n_splits=splits, impl=impl)
+                        scale=scale, gate=gate.reshape(B * T, H).cuda(), workspace=ws, n_splits=splits, impl=impl,
+                        status=status)
+        assert int(status) == 0
         want = torch.stack([plain_latent_attention(q[b].double(), data[b].double(), gate[b].double(), lens[b], window, scale) for b in range(B)])
         close(out.view(B, T, H, r), want, dtype, f32=3e-5)
 
