@@ -1,4 +1,4 @@
-// Latent attention on tcgen05 (sm_100a): one persistent CTA per SM walks through (query row, head group, key split)
+// Latent attention on tcgen05 (sm_100a): one or two persistent CTAs per SM walk through (query row, head group, key split)
 // items; the latents of an item pass through shared memory once and serve all its heads, as keys and as values.
 //
 // A tile is 128 latents x r columns, cut into units of 128 columns (two 64-column, 128-byte-swizzled blocks, 32 KB).
@@ -94,6 +94,26 @@ __device__ __forceinline__ void tmem_ld16_nowait(uint32_t addr, float* v) {
       : "r"(addr)
       : "memory");
 }
+// Eight MMAs over one unit in a single statement with constant descriptor steps.  Offsets in 16-byte units: A advances by
+// A_STEP, B by 2 (16 elements along its 128-byte rows); the second four start at A_HALF and B_HALF.  The first MMA takes
+// the accumulate flag.
+template <int A_STEP, int A_HALF, int B_HALF>
+__device__ __forceinline__ void lt_mma8(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p0, pt;\n\t.reg .b64 a, b;\n\t"
+      "setp.ne.b32 p0, %4, 0;\n\tsetp.eq.b32 pt, 0, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p0;\n\t"
+      "add.u64 a, %1, %5;\n\tadd.u64 b, %2, 2;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %6;\n\tadd.u64 b, %2, 4;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %7;\n\tadd.u64 b, %2, 6;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %8;\n\tadd.u64 b, %2, %12;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %9;\n\tadd.u64 b, %2, %13;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %10;\n\tadd.u64 b, %2, %14;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %11;\n\tadd.u64 b, %2, %15;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP), "n"(A_HALF), "n"(A_HALF + A_STEP),
+      "n"(A_HALF + 2 * A_STEP), "n"(A_HALF + 3 * A_STEP), "n"(B_HALF), "n"(B_HALF + 2), "n"(B_HALF + 4), "n"(B_HALF + 6)
+      : "memory");
+}
 // The four softmax warps: a barrier, and a barrier that tells every thread whether any of them said yes.
 __device__ __forceinline__ void lt_sync() { asm volatile("barrier.sync 1, 128;" ::: "memory"); }
 __device__ __forceinline__ bool lt_any(bool mine) {
@@ -135,7 +155,7 @@ __device__ __forceinline__ float lt_reduce16(const float* v, int lane, F op) {
 }
 
 template <int NB>  // heads per group = 16 NB
-__global__ void __launch_bounds__(kLtThreads, 1)
+__global__ void __launch_bounds__(kLtThreads, NB == 4 ? 1 : 2)
 latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc, const LtParams p) {
   constexpr int N = 16 * NB;
   constexpr uint32_t kIdescS = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | (8u << 24);
@@ -148,8 +168,13 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   const int U = p.upt, NU = p.n_units;
   uint8_t* sU = smem;
   uint8_t* sQ = sU + (size_t)NU * kLtUnit;
-  uint8_t* sP = sQ + (size_t)2 * U * kQBlock;  // two buffers of two blocks
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 4 * kPBlock);
+  uint8_t* sP = sQ + (size_t)2 * U * kQBlock;  // one or two buffers of two blocks
+  // With room for two tiles in the ring the scores of the next tile are issued before the sums of this one, and P needs
+  // two buffers; otherwise the next scores follow the sums, and their arrival also says that P has been read.  (Issuing
+  // the part of the next scores that the ring could hold before the sums was measured 12 % slower: every change between
+  // the two kinds of product costs the tensor pipe more than the wait it fills.)
+  const bool ahead = NU >= 2 * U;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + (ahead ? 4 : 2) * kPBlock);
   float* red = reinterpret_cast<float*>(bars + 32);  // [4 warps][N]
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(red + 4 * N);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -225,7 +250,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   } else if (warp == 4) {
     // ================= MMA issuer =================
     if (lane == 0) {
-      const bool ahead = NU >= 2 * U;
+      const uint64_t dC = smem_desc(0, 16, 1024), dM = smem_desc(0, kLtBlock, 1024);  // K-major rows; MN-major pairs of blocks
       unsigned un = 0u, g = 0u, items = 0u;  // units whose scores have been issued; tiles; items
       unsigned uo = 0u;                      // units whose sums have been issued
       bool ok = true;
@@ -240,12 +265,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
             ok = wait_or_abort(bar_u + 8 * s, (un / (unsigned)NU) & 1u, abort_flag, 53);
             if (!ok) return;
             tc_fence_after();
-#pragma unroll
-            for (int ks = 0; ks < 8; ++ks) {
-              const uint32_t ca = aU + s * kLtUnit + (ks >> 2) * kLtBlock + (ks & 3) * 32;
-              const uint32_t cq = aQ + (2 * u + (ks >> 2)) * kQBlock + (ks & 3) * 32;
-              umma_ss(d, smem_desc(ca, 16, 1024), smem_desc(cq, 16, 1024), kIdescS, (u > 0 || ks > 0) ? 1u : 0u);
-            }
+            lt_mma8<2, kLtBlock / 16, kQBlock / 16>(d, dC + ((aU + s * kLtUnit) >> 4), dC + ((aQ + 2 * u * kQBlock) >> 4), kIdescS, u > 0 ? 1u : 0u);
           }
           umma_commit(bar_s + 8 * (gt & 1u));
           if (last) umma_commit(bar_qf);
@@ -260,12 +280,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
           tc_fence_after();
           for (int u = 0; u < U; ++u, ++uo) {
             const unsigned s = uo % (unsigned)NU;
-#pragma unroll
-            for (int ks = 0; ks < 8; ++ks) {
-              const uint32_t pa = aP + (2 * b + (ks >> 2)) * kPBlock + (ks & 3) * 32;
-              umma_ss(tmem + 2 * N + u * N, smem_desc(aU + s * kLtUnit + ks * 2048, kLtBlock, 1024), smem_desc(pa, 16, 1024), kIdescO,
-                      (j > 0 || ks > 0) ? 1u : 0u);
-            }
+            lt_mma8<128, 512, kPBlock / 16>(tmem + 2 * N + u * N, dM + ((aU + s * kLtUnit) >> 4), dC + ((aP + (ahead ? 2 * b * kPBlock : 0u)) >> 4),
+                                            kIdescO, j > 0 ? 1u : 0u);
             umma_commit(bar_uf + 8 * s);
           }
           umma_commit(bar_o + 8 * b);
@@ -361,7 +377,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
           }
           lt_sync();  // `red` may be written again
         }
-        uint8_t* pb = sP + (2 * b + (tid >> 6)) * kPBlock + (tid & 7) * 2;
+        uint8_t* pb = sP + ((ahead ? 2 * b : 0u) + (tid >> 6)) * kPBlock + (tid & 7) * 2;
         const int chunk = (tid & 63) >> 3;
 #pragma unroll
         for (int h = 0; h < N; ++h) {
@@ -462,12 +478,13 @@ static bool encode_3d(CUtensorMap* map, const void* base, const cuuint64_t (&dim
 
 // heads per group, and what fits beside Q and P in the shared memory (limit: opt-in bytes per CTA)
 static int lt_heads(int H) { return H <= 16 ? 16 : (H <= 32 ? 32 : 64); }
-static size_t lt_fixed_bytes(int N, int U) { return (size_t)2 * U * N * 128 + (size_t)4 * N * 128 + 256 + (size_t)16 * N + 64 + 1024; }
+static size_t lt_bytes(int N, int U, int units) {
+  return (size_t)2 * U * N * 128 + (size_t)(units >= 2 * U ? 4 : 2) * N * 128 + 256 + (size_t)16 * N + 64 + 1024 + (size_t)units * kLtUnit;
+}
 static int lt_units(int N, int U, size_t limit) {
-  const size_t fixed = lt_fixed_bytes(N, U);
-  if (fixed >= limit) return 0;
-  const int n = (int)((limit - fixed) / kLtUnit);
-  return n > kLtMaxUnits ? kLtMaxUnits : n;
+  int n = kLtMaxUnits;
+  while (n > 0 && lt_bytes(N, U, n) > limit) --n;
+  return n;
 }
 
 template <int NB>
@@ -518,7 +535,17 @@ int latent_tc_launch(const LatentArgs& a, const dgpt_kv_layout& kv, cudaStream_t
   p.n_groups = (a.H + N - 1) / N;
   p.n_items = p.n_rows * p.n_groups * a.n_splits;
   p.upt = (a.r + 127) / 128;
+  // Two CTAs per SM where half the shared memory holds a tile and a unit: while one waits for its scores or its
+  // probabilities, the other has products to run.  (NB = 4 needs the registers of a whole SM.)
+  int per_sm = 1;
   p.n_units = lt_units(N, p.upt, (size_t)limit);
+  if (N < 64 && p.n_items > sms) {
+    const int half = lt_units(N, p.upt, (size_t)(limit - 1024) / 2);  // each CTA costs another KB of the SM's 228
+    if (half > p.upt) {
+      per_sm = 2;
+      p.n_units = half;
+    }
+  }
   const int pt = kv.page_tokens;
   p.box = kv.page_table && pt < kLtKeys ? pt : kLtKeys;
   p.align = kv.page_table ? p.box : 1;  // a dense run may be entered at any slot
@@ -536,8 +563,8 @@ int latent_tc_launch(const LatentArgs& a, const dgpt_kv_layout& kv, cudaStream_t
     const cuuint32_t box[3] = {64, (cuuint32_t)p.box, 1};
     if (!encode_3d(&mc, kv.k_base, dims, strides, box)) return DGPT_E_CUDA;
   }
-  const size_t smem = lt_fixed_bytes(N, p.upt) + (size_t)p.n_units * kLtUnit;
-  const int grid = p.n_items < sms ? p.n_items : sms;
+  const size_t smem = lt_bytes(N, p.upt, p.n_units);
+  const int grid = p.n_items < per_sm * sms ? p.n_items : per_sm * sms;
   if (N == 16) return lt_launch<1>(mq, mc, p, grid, smem, st);
   if (N == 32) return lt_launch<2>(mq, mc, p, grid, smem, st);
   return lt_launch<4>(mq, mc, p, grid, smem, st);
