@@ -176,7 +176,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   const bool ahead = NU >= 2 * U;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + (ahead ? 4 : 2) * kPBlock);
   float* red = reinterpret_cast<float*>(bars + 32);  // [4 warps][N]
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(red + 4 * N);
+  float* fac = red + 4 * N;                          // [4 warps][N]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(fac + 4 * N);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   const uint32_t aU = smem_u32(sU), aQ = smem_u32(sQ), aP = smem_u32(sP);
   const uint32_t bar0 = smem_u32(bars);
@@ -305,6 +306,15 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
     for (int item = blockIdx.x; item < p.n_items; item += gridDim.x) {
       const LtItem it = lt_item(p, item, N);
       const int nh = min(N, p.a.H - it.h0);
+      constexpr int HL = (N + 31) / 32;  // heads a lane looks after at the end of the item
+      float gate[HL];
+#pragma unroll
+      for (int c = 0; c < HL; ++c) {  // wanted at the end only
+        const int h = lane + 32 * c;
+        gate[c] = 1.f;
+        if (p.a.gate && h < nh)
+          gate[c] = __bfloat162float(static_cast<const __nv_bfloat16*>(p.a.gate)[(long long)it.row * p.a.gate_rs + it.h0 + h]);
+      }
       float m[N], l[N];
 #pragma unroll
       for (int h = 0; h < N; ++h) {
@@ -402,52 +412,60 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         if (lane < 16) red[warp * N + 16 * c + lane] = t;
       }
       lt_sync();
-      float f[N];  // 1 / sum and gate, or the sum itself for a split
-#pragma unroll
-      for (int h = 0; h < N; ++h) {
-        const float sum = (red[h] + red[N + h]) + (red[2 * N + h] + red[3 * N + h]);
-        f[h] = sum;
-        if (p.a.n_splits == 1) {
-          f[h] = sum > 0.f ? 1.f / sum : 0.f;
-          if (p.a.gate && h < nh)
-            f[h] *= 1.f / (1.f + __expf(-__bfloat162float(static_cast<const __nv_bfloat16*>(p.a.gate)[(long long)it.row * p.a.gate_rs + it.h0 + h])));
-        }
-      }
-      lt_sync();
       const long long rh0 = (long long)it.row * p.a.H + it.h0;
       const long long slot0 = (long long)it.split * RH + rh0;
-      if (p.a.n_splits > 1 && tid == 0) {
+      // lane h: 1 / sum and gate of head h, or the sum itself for a split
 #pragma unroll
-        for (int h = 0; h < N; ++h) {
-          if (h < nh) {
-            p.a.ws_ml[2 * (slot0 + h)] = m[h];
-            p.a.ws_ml[2 * (slot0 + h) + 1] = f[h];
-          }
+      for (int c = 0; c < HL; ++c) {
+        const int h = lane + 32 * c;
+        if (h < N) {
+          const float sum = (red[h] + red[N + h]) + (red[2 * N + h] + red[3 * N + h]);
+          float f = sum > 0.f ? 1.f / sum : 0.f;
+          if (p.a.gate) f *= 1.f / (1.f + __expf(-gate[c]));
+          fac[warp * N + h] = f;
+          if (p.a.n_splits > 1 && warp == 0 && h < nh) p.a.ws_ml[2 * (slot0 + h) + 1] = sum;
         }
       }
-      for (int u = 0; u < U && it.n > 0; ++u) {
-        const int col = u * 128 + tid;
+      if (p.a.n_splits > 1 && tid == 0) {
 #pragma unroll
-        for (int c = 0; c < NB; ++c) {
-          float v[16];
-          tmem_ld16_nowait(lane_addr + 2 * N + u * N + c * 16, v);
-          tc_wait_ld();
-          if (col < p.a.r) {
+        for (int h = 0; h < N; ++h)
+          if (h < nh) p.a.ws_ml[2 * (slot0 + h)] = m[h];
+      }
+      lt_sync();  // `red` may be written again, `fac` is complete
+      if (it.n > 0) {
+        for (int u = 0; u < U; ++u) {
+          const int col = u * 128 + tid;
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-              const int h = 16 * c + i;
-              if (h >= nh) continue;
-              if (p.a.n_splits > 1) p.a.ws_o[(slot0 + h) * p.a.r + col] = v[i];
-              else
-                static_cast<__nv_bfloat16*>(p.a.out)[(long long)it.row * p.a.out_rs + (long long)(it.h0 + h) * p.a.r + col] =
-                    __float2bfloat16_rn(v[i] * f[h]);
+          for (int c = 0; c < NB; ++c) {
+            float v[16];
+            tmem_ld16_nowait(lane_addr + 2 * N + u * N + c * 16, v);
+            tc_wait_ld();
+            if (u == U - 1 && c == NB - 1) {
+              tc_fence_before();
+              mbar_arrive(bar_of);  // the next item may overwrite O
+            }
+            if (p.a.n_splits > 1) {
+              if (col < p.a.r) {
+#pragma unroll
+                for (int i = 0; i < 16; ++i)
+                  if (16 * c + i < nh) p.a.ws_o[(slot0 + 16 * c + i) * p.a.r + col] = v[i];
+              }
+              continue;
+            }
+            // two columns of one head per store: an even lane takes the even head of a pair, its neighbour the odd one
+            // (r is a multiple of 8, so both columns exist or neither does)
+            const bool odd = lane & 1;
+            __nv_bfloat16* dst = static_cast<__nv_bfloat16*>(p.a.out) + (long long)it.row * p.a.out_rs + (long long)it.h0 * p.a.r + (col & ~1);
+#pragma unroll
+            for (int i = 0; i < 16; i += 2) {
+              const float x = v[i] * fac[warp * N + 16 * c + i], y = v[i + 1] * fac[warp * N + 16 * c + i + 1];
+              const float got = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
+              const int h = 16 * c + i + (odd ? 1 : 0);
+              if (h < nh && col < p.a.r)
+                *reinterpret_cast<__nv_bfloat162*>(dst + (long long)h * p.a.r) = odd ? __floats2bfloat162_rn(got, y) : __floats2bfloat162_rn(x, got);
             }
           }
         }
-      }
-      if (it.n > 0) {
-        tc_fence_before();
-        mbar_arrive(bar_of);
       } else if (p.a.n_splits == 1) {  // no keys at all
         for (int u = 0; u < U; ++u) {
           const int col = u * 128 + tid;
@@ -479,7 +497,7 @@ static bool encode_3d(CUtensorMap* map, const void* base, const cuuint64_t (&dim
 // heads per group, and what fits beside Q and P in the shared memory (limit: opt-in bytes per CTA)
 static int lt_heads(int H) { return H <= 16 ? 16 : (H <= 32 ? 32 : 64); }
 static size_t lt_bytes(int N, int U, int units) {
-  return (size_t)2 * U * N * 128 + (size_t)(units >= 2 * U ? 4 : 2) * N * 128 + 256 + (size_t)16 * N + 64 + 1024 + (size_t)units * kLtUnit;
+  return (size_t)2 * U * N * 128 + (size_t)(units >= 2 * U ? 4 : 2) * N * 128 + 256 + (size_t)32 * N + 64 + 1024 + (size_t)units * kLtUnit;
 }
 static int lt_units(int N, int U, size_t limit) {
   int n = kLtMaxUnits;
