@@ -927,6 +927,8 @@ def kernel_case(name: str, iters: int = 8) -> None:
     depthmix:    config-4 rows, 8 candidates (mid-stack).
     fmha_prefix: shared-prompt phase of a config-4 decode step (4096 rows x 1024 prompt keys, 12 heads x 64).
     linear:      first feed-forward GEMM of a config-4 decode step with the SwiGLU epilogue.
+    latent_attn: decode attention on cached latents, 296 rows x 16 heads x 1024 keys of 256 numbers.
+    fmha_window: prefill attention with a window of 1024, 8192 tokens, 16 heads of 128.
     Prints one JSON line with the CUDA-event time per launch and the achieved rate.
     """
     from diff_gpt_b200 import ops
@@ -1006,6 +1008,38 @@ def kernel_case(name: str, iters: int = 8) -> None:
             ops.linear(a, wgt, act, swiglu=(1.702, 7.0), status=st)
 
         work = 2 * M * N * K
+        unit, peak = "TFLOP/s", pk["bf16_tflops"]
+    elif name == "latent_attn":
+        # one decode step of a latent-attention layer: 296 rows, 16 heads on 1024 latents of 256 numbers (155 MB)
+        R, H, r, W, pt = 296, 16, 256, 1024, 64
+        pool = torch.randn((R * W // pt, pt, r), device=dev, dtype=torch.bfloat16, generator=g)
+        table = torch.randperm(R * W // pt, device=dev, generator=g).to(torch.int32).view(R, W // pt)
+        lay = ops.kv_layout(pool, pool, pt * r, 0, pt, table, n_pages=R * W // pt)
+        q = torch.randn((R, H * r), device=dev, dtype=torch.bfloat16, generator=g)
+        gate = torch.randn((R, H), device=dev, dtype=torch.bfloat16, generator=g)
+        o = torch.empty_like(q)
+        zero, n1 = torch.zeros(R, dtype=torch.int32, device=dev), torch.full((R,), W, dtype=torch.int32, device=dev)
+        st = torch.zeros(1, dtype=torch.int32, device=dev)
+
+        def launch():
+            ops.latent_attn(q, lay, None, zero, n1, None, o, n_seq=R, T=1, H=H, r=r, window=W, scale=0.0884, gate=gate, status=st)
+
+        work = R * (W * r + 2 * H * r + H) * 2
+        unit, peak = "GB/s", pk["hbm_gbs"]
+    elif name == "fmha_window":
+        # windowed prefill attention: 8192 tokens, 16 heads of 128, window 1024
+        T, H, D, W = 8192, 16, 128, 1024
+        q = torch.randn((T, H * D), device=dev, dtype=torch.bfloat16, generator=g)
+        kv = torch.randn((T, 2 * H * D), device=dev, dtype=torch.bfloat16, generator=g)
+        gate = torch.randn((T, H), device=dev, dtype=torch.bfloat16, generator=g)
+        o = torch.empty_like(q)
+        st = torch.zeros(1, dtype=torch.int32, device=dev)
+
+        def launch():
+            ops.fmha_window(q, kv[:, : H * D], kv[:, H * D :], o, B=1, H=H, D=D, n_keys=T, q_offset=0, window=W, scale=D**-0.5,
+                            gate=gate, status=st)
+
+        work = 4 * D * H * (T * W - W * (W - 1) // 2)
         unit, peak = "TFLOP/s", pk["bf16_tflops"]
     elif name == "sample":
         R, V = TRAJECTORIES, CFG4["vocab_size"]
@@ -1254,6 +1288,13 @@ def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
     report("gpt.fmha_prefill", lambda: ops.fmha_prefill(q, lay, o, B=1, H=H, Tq=T, D=Dg, q_batch_stride=T * C, q_row_stride=C,
                                                         o_batch_stride=T * C, o_row_stride=C, kv_len_all=T, causal=True, status=st),
            8, None, 4 * Dg * H * (T * (T + 1) // 2))
+    S = 2 * W  # causal over 2 W keys: W per query on average, as the window has
+    B = max(1, T // S)
+    kvs = rnd(B, 2, H, S, Dg)
+    lays = ops.kv_layout(kvs[0, 0], kvs[0, 1], 2 * H * S * Dg, S * Dg, S)
+    report("gpt.fmha_prefill_2W", lambda: ops.fmha_prefill(q, lays, o, B=B, H=H, Tq=S, D=Dg, q_batch_stride=S * C, q_row_stride=C,
+                                                           o_batch_stride=S * C, o_row_stride=C, kv_len_all=S, causal=True, status=st),
+           8, None, B * 4 * Dg * H * (S * (S + 1) // 2))
     cands = [rnd(T, C) for _ in range(terms)]
     wq = rnd(C)
     report("gpt.depthmix", lambda: ops.depthmix(cands, wq, None, u), 8, T * C * 2 * (terms + 1))
@@ -1296,7 +1337,7 @@ def run_design(args) -> None:
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernel-case", default=None, choices=["decode_attn", "fmha", "fmha_long", "fmha_pair", "sample", "depthmix", "fmha_prefix", "linear"],
+    ap.add_argument("--kernel-case", default=None, choices=["decode_attn", "fmha", "fmha_long", "fmha_pair", "sample", "depthmix", "fmha_prefix", "linear", "latent_attn", "fmha_window"],
                     help="run one kernel alone on a small case (for ncu) and exit")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=3)
