@@ -204,33 +204,41 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(const LatentAr
   }
 }
 
-// One warp per (row, head): every lane knows the weights of all splits, then the columns are summed over the splits.
+// CTA per (row, head): the splits' weights once in shared memory, then one thread per column.
+constexpr int kLatMaxSplits = 256;
 template <typename T>
-__global__ void latent_combine_kernel(const LatentArgs a) {
+__global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a) {
+  __shared__ float wt[kLatMaxSplits];
+  __shared__ float scratch[40];
   const long long RH = (long long)a.n_seq * a.Tn * a.H;
-  const long long rh = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-  if (rh >= RH) return;
-  const int lane = threadIdx.x & 31;
+  const long long rh = blockIdx.x;
   const long long row = rh / a.H;
-  const int h = (int)(rh - row * a.H);
+  const int h = (int)(rh - row * a.H), tid = threadIdx.x, n = a.n_splits;
   float m = -INFINITY;
-  for (int s = lane; s < a.n_splits; s += 32) m = fmaxf(m, a.ws_ml[2 * (s * RH + rh)]);
-  m = warp_max(m);
+  for (int s = tid & 31; s < n; s += 32) m = fmaxf(m, a.ws_ml[2 * (s * RH + rh)]);
+  m = warp_max(m);  // the same in every warp
   float l = 0.f;
-  for (int s = lane; s < a.n_splits; s += 32) {
+  for (int s = tid; s < n; s += 128) {
     const float ms = a.ws_ml[2 * (s * RH + rh)];
-    l += ms == -INFINITY ? 0.f : a.ws_ml[2 * (s * RH + rh) + 1] * exp2f(ms - m);
+    const float e = ms == -INFINITY ? 0.f : exp2f(ms - m);
+    wt[s] = e;
+    l += e == 0.f ? 0.f : a.ws_ml[2 * (s * RH + rh) + 1] * e;
   }
-  l = warp_sum(l);
+  l = block_sum(l, scratch);  // and `wt` is complete
   float f = l > 0.f ? 1.f / l : 0.f;
   if (a.gate) f *= 1.f / (1.f + expf(-Io<T>::ld(static_cast<const T*>(a.gate) + row * a.gate_rs + h)));
   T* dst = static_cast<T*>(a.out) + row * a.out_rs + (long long)h * a.r;
-  for (int c = lane; c < a.r; c += 32) {
+  for (int c = tid; c < a.r; c += 128) {
     float acc = 0.f;
-    for (int s = 0; s < a.n_splits; ++s) {
-      const float ms = a.ws_ml[2 * (s * RH + rh)];
-      if (ms != -INFINITY) acc += a.ws_o[(s * RH + rh) * a.r + c] * exp2f(ms - m);
+    int s = 0;
+    for (; s + 8 <= n; s += 8) {  // eight loads in flight; a split without keys has weight 0 and holds nothing
+      float v[8];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) v[u] = a.ws_o[((s + u) * RH + rh) * a.r + c];
+#pragma unroll
+      for (int u = 0; u < 8; ++u) acc += wt[s + u] == 0.f ? 0.f : wt[s + u] * v[u];
     }
+    for (; s < n; ++s) acc += wt[s] == 0.f ? 0.f : wt[s] * a.ws_o[(s * RH + rh) * a.r + c];
     Io<T>::st(dst + c, acc * f);
   }
 }
@@ -317,7 +325,8 @@ extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_
                                 int32_t window, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
   DGPT_REQUIRE(q && out && start1 && len1, "latent_attn: NULL pointer");
   DGPT_REQUIRE(n_seq >= 0 && T >= 0 && H > 0 && r > 0 && r % 8 == 0 && window >= 0, "latent_attn: bad sizes");
-  DGPT_REQUIRE(n_splits >= 1 && n_splits <= 65535 && H <= 65535, "latent_attn: bad number of splits or heads");
+  DGPT_REQUIRE(n_splits >= 1 && n_splits <= kLatMaxSplits && H <= 65535,
+               "latent_attn: 1 to %d splits", kLatMaxSplits);
   DGPT_REQUIRE(impl >= 0 && impl <= 2, "latent_attn: impl must be 0 (auto), 1 (CUDA cores) or 2 (tcgen05)");
   DGPT_REQUIRE(dtype == DGPT_F32 || dtype == DGPT_BF16, "latent_attn: unknown dtype %d", dtype);
   DGPT_REQUIRE((reinterpret_cast<uintptr_t>(q) & 15) == 0 && q_row_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
@@ -356,8 +365,7 @@ extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_
   else e = latent_simt_launch<__nv_bfloat16>(a, st);
   if (e || n_splits == 1) return e;
   const long long RH = R * H;
-  const unsigned grid = (unsigned)((RH + 7) / 8);
-  if (dtype == DGPT_F32) latent_combine_kernel<float><<<grid, 256, 0, st>>>(a);
-  else latent_combine_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>(a);
+  if (dtype == DGPT_F32) latent_combine_kernel<float><<<(unsigned)RH, 128, 0, st>>>(a);
+  else latent_combine_kernel<__nv_bfloat16><<<(unsigned)RH, 128, 0, st>>>(a);
   return launch_status("latent_combine");
 }

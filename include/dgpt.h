@@ -368,7 +368,7 @@ int dgpt_latent_append(const void* in, int64_t in_row_stride, const float* w, fl
  * row = s * T + t.  Row (s, t) sees the last `window` (0 = all) of the keys 0 .. n-1, n = len0[s] + len1[s] + step + t,
  * where key i is slot i for i < len0[s] and slot start1[s] + i - len0[s] from there on (len0 NULL = 0).
  * q, out: device [n_seq*T, H*r] with row strides; gate: [n_seq*T, H] in dtype or NULL; r a multiple of 8.
- * n_splits > 1 splits each row's keys over CTAs (workspace from the _bytes call with R = n_seq * T, 16-byte aligned).
+ * n_splits > 1 (at most 256) splits each row's keys over CTAs (workspace from the _bytes call with R = n_seq * T, 16-byte aligned).
  * impl: 0 = choose, 1 = CUDA cores (any r), 2 = tcgen05 (bf16, r <= 512, a dense run of slots per sequence or pages of 8 to
  * 64 or a multiple of 128 tokens) or fail.  status: device int32, set non-zero if a bounded wait ran out. */
 size_t dgpt_latent_attn_workspace_bytes(int32_t R, int32_t H, int32_t r, int32_t n_splits);
