@@ -12,12 +12,13 @@ from . import _lib  # noqa: F401  (raises if the shared object is missing)
 from .model.delunex import Delunex
 from .model.engine import Engine, StepRunner
 from .model.gpt import GPT, BaseGPT
-from .model.kv_cache import KVCache, LatentCache, PagedKVCache
+from .model.kipolix import Kipolix
+from .model.kv_cache import KVCache, LatentCache, PagedKVCache, RowCache
 from .model.registry import load_model
 from .sampler.nucleus import NucleusSampler
 from .sampler.sampler import Sampler
 from .sampler.temperature import TemperatureSampler
 
 __all__ = [
-    "GPT", "BaseGPT", "Delunex", "KVCache", "LatentCache", "PagedKVCache", "Engine", "StepRunner", "load_model", "Sampler", "TemperatureSampler", "NucleusSampler",
+    "GPT", "BaseGPT", "Delunex", "Kipolix", "KVCache", "LatentCache", "PagedKVCache", "RowCache", "Engine", "StepRunner", "load_model", "Sampler", "TemperatureSampler", "NucleusSampler",
 ]

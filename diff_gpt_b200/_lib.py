@@ -99,6 +99,32 @@ PROTOTYPES = {
         C.c_int,
         [_p, _i64, _kvp, _p, _p, _p, _p, _p, _i64, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32, _p, _p],
     ),
+    "dgpt_fmha_grouped": (
+        C.c_int,
+        [_p, _i64, _i64, _kvp, _i64, _i32, _p, _i64, _i64, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _f32, _i32, _i32, _p, _p],
+    ),
+    "dgpt_grouped_attn": (
+        C.c_int,
+        [_p, _i64, _kvp, _i32, _i32, _p, _p, _p, _p, _p, _i64, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32, _i32,
+         _f32, _i32, _i32, _p, _p],
+    ),
+    "dgpt_silu_mul": (C.c_int, [_p, _p, _i64, _i32, _p]),
+    "dgpt_embed_streams": (
+        C.c_int, [_p, _p, _p, _p, _i32, _p, _i64, _i64, _i64, _p, _i32, _p, _f32, _p, _p, _i32, _i32, _i32, _i32, _p]
+    ),
+    "dgpt_streams_step": (C.c_int, [_p, _i64, _p, _p, _p, _p, _i32, _p, _f32, _p, _i64, _p, _i64, _i32, _i32, _p]),
+    "dgpt_streams_final": (C.c_int, [_p, _i64, _p, _p, _p, _i32, _p, _f32, _p, _p, _i64, _i64, _i32, _i32, _p]),
+    "dgpt_proj_norm_rope_append": (
+        C.c_int,
+        [_p, _i64, _p, _p, _i32, _i32, _f32, _p, _i32, _i32, _p, _i64, _kvp, _i32, _p, _p, _p, _i32, _i32, _i32, _i32, _i32, _i32,
+         _i32, _p, _p],
+    ),
+    "dgpt_retention_workspace_bytes": (_sz, [_i32, _i32, _i32, _i32, _i32]),
+    "dgpt_retention": (
+        C.c_int,
+        [_p, _i64, _i32, _i32, _i32, _i32, _p, _i32, _i32, _p, _p, _p, _f32, _p, _p, _f32, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32,
+         _i32, _i32, _i32, _p, _p],
+    ),
     "dgpt_embed_scale": (C.c_int, [_p, _p, _p, _i64, _i32, _i32, _f32, _i32, _p]),
     "dgpt_norm_add": (C.c_int, [_p, _p, _f32, _p, _p, _p, _i64, _i32, _i32, _p]),
     "dgpt_depth_avg_conv": (C.c_int, [_p, _i64, _i32, _p, _p, _i32, _p, _p, _p, _p, _i32, _i32, _i32, _i32, _p]),
@@ -108,7 +134,7 @@ PROTOTYPES = {
 }
 _NOT_LAUNCHING = {
     "dgpt_last_error", "dgpt_version", "dgpt_decode_attn_workspace_bytes", "dgpt_decode_attn_static_capacity_bytes",
-    "dgpt_lmhead_workspace_bytes", "dgpt_latent_attn_workspace_bytes",
+    "dgpt_lmhead_workspace_bytes", "dgpt_latent_attn_workspace_bytes", "dgpt_retention_workspace_bytes",
 }
 
 

@@ -23,6 +23,8 @@ struct FmhaArgs {
   int window = 0;           // query i sees keys (q_offset + i - window, q_offset + i]; 0 = all of them (causal only)
   float scale = 0.f;        // score scale; 0 = 1 / sqrt(D)
   long long kv_ts = 0;      // elements between consecutive keys of a head; 0 = D
+  int kv_heads = 0;         // key/value heads; query head h reads h / (H / kv_heads); 0 = H
+  int keep_first = 0;       // with a window: keys j < keep_first are seen from every distance
   const void* hgate = nullptr;  // [B * Tq, H] in dtype: output of head h is multiplied by sigmoid(hgate)
   long long hgate_rs = 0;
 };
@@ -45,6 +47,8 @@ struct TcParams {
   int d_head;        // head_dim of the tensors in global memory (32 rides on the 64-wide kernels: the TMA boxes are 64 wide
                      // and the columns past the tensor's extent arrive as zeros, so scores and outputs are unchanged)
   int window;        // 0 = no lower bound
+  int keep_first;    // keys below this are seen whatever the window
+  int kv_div;        // query heads per key/value head
   const void* hgate; // bf16 [B * Tq, H], or NULL
   long long hgate_rs;
   int BH, group_bh;  // two-query-tile kernel: (batch, head) pairs in all, and how many are worked on at a time
@@ -56,10 +60,16 @@ __device__ __forceinline__ float head_gate(const void* hgate, long long rs, long
   if (hgate == nullptr) return 1.f;
   return 1.f / (1.f + expf(-Io<T>::ld(static_cast<const T*>(hgate) + row * rs + h)));
 }
-// First key tile of `tile` keys that a query at position `first_q` (the tile's lowest) can see.
+// First key tile of `tile` keys inside the window of a query at position `first_q` (the query tile's lowest).
 __device__ __forceinline__ int window_first_tile(int window, int first_q, int tile) {
   return window > 0 ? max(0, first_q - window + 1) / tile : 0;
 }
+// Key tiles ahead of that one that hold kept first keys.  A query tile visits tiles [0, n_kept) and then those from
+// `tile0` on: its j-th tile is tile_of(j).
+__device__ __forceinline__ int kept_tiles(int keep_first, int tile0, int tile) {
+  return min(tile0, (keep_first + tile - 1) / tile);
+}
+__device__ __forceinline__ int tile_of(int j, int n_kept, int tile0) { return j < n_kept ? j : tile0 + (j - n_kept); }
 
 // warp-level kernel (fmha_simt.cu)
 int fmha_simt(const FmhaArgs& a, const KvView& kv, cudaStream_t st);

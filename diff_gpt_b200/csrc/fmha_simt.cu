@@ -20,7 +20,7 @@ __global__ void __launch_bounds__(128)
 fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView kv, const int* __restrict__ kv_len,
                  int kv_len_all, void* __restrict__ o, long long o_bs, long long o_rs, int o_f32,
                  float* __restrict__ lse, int H, int Tq, int q_offset, int causal, float scale_log2, int window,
-                 const void* __restrict__ hgate, long long hgate_rs) {
+                 int keep_first, int kv_div, const void* __restrict__ hgate, long long hgate_rs) {
   constexpr int DP = D / SPLIT;       // elements per thread
   constexpr int BM = 128 / SPLIT;     // queries per CTA
   constexpr int VEC = Io<T>::kVec16;
@@ -59,7 +59,10 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
   const T* kbase = static_cast<const T*>(kv.k);
   const T* vbase = static_cast<const T*>(kv.v);
 
-  for (int j0 = window_first_tile(window, q_offset + q0, kSimtBN) * kSimtBN; j0 < kmax; j0 += kSimtBN) {
+  const int tile0 = window_first_tile(window, q_offset + q0, kSimtBN), n_kept = kept_tiles(keep_first, tile0, kSimtBN);
+  for (int tile = 0;; ++tile) {
+    const int j0 = tile_of(tile, n_kept, tile0) * kSimtBN;
+    if (j0 >= kmax) break;
     __syncthreads();
     constexpr int VPR = D / VEC;  // 16-byte vectors per key row
     for (int idx = tid; idx < kSimtBN * VPR; idx += 128) {
@@ -67,7 +70,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
       const int slot = j0 + tk;
       float kf[VEC], vf[VEC];
       if (slot < klen) {
-        const long long off = kv_offset(kv, b, h, slot, D) + pv * VEC;
+        const long long off = kv_offset(kv, b, h / kv_div, slot, D) + pv * VEC;
         ld16<T>(kbase + off, kf);
         ld16<T>(vbase + off, vf);
       } else {
@@ -97,7 +100,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
 #pragma unroll
         for (int x = 1; x < SPLIT; x <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, x);
         const int j = j0 + kb + kk;
-        s[kk] = (q_ok && j < klen && j <= my_last && j >= my_first) ? dot : -INFINITY;
+        s[kk] = (q_ok && j < klen && j <= my_last && (j >= my_first || j < keep_first)) ? dot : -INFINITY;
         smax = fmaxf(smax, s[kk]);
       }
       if (smax == -INFINITY) continue;  // nothing visible in this group (no shuffles below)
@@ -150,7 +153,9 @@ static int fmha_simt_launch(const FmhaArgs& a, const KvView& kv, cudaStream_t st
   const float scale_log2 = a.scale > 0.f ? a.scale * kLog2e : kLog2e / sqrtf((float)D);
   fmha_simt_kernel<T, D, SPLIT><<<grid, 128, 0, st>>>(static_cast<const T*>(a.q), a.q_bs, a.q_rs, kv, a.kv_len,
                                                       a.kv_len_all, a.o, a.o_bs, a.o_rs, a.o_f32, a.lse, a.H, a.Tq,
-                                                      a.q_offset, a.causal, scale_log2, a.window, a.hgate, a.hgate_rs);
+                                                      a.q_offset, a.causal, scale_log2, a.window,
+                                                      a.window > 0 ? a.keep_first : 0, a.kv_heads > 0 ? a.H / a.kv_heads : 1, a.hgate,
+                                                      a.hgate_rs);
   return launch_status("fmha_simt");
 }
 
@@ -222,26 +227,22 @@ extern "C" int dgpt_fmha_prefill(const void* q, int64_t q_batch_stride, int64_t 
   return fmha_simt(a, view, st);
 }
 
-extern "C" int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const void* k, const void* v,
-                                int64_t kv_batch_stride, int64_t kv_row_stride, int64_t kv_head_stride, int32_t n_keys, void* o,
-                                int64_t o_batch_stride, int64_t o_row_stride, const void* gate, int64_t gate_row_stride,
-                                int32_t B, int32_t H, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, float scale,
-                                int32_t dtype, int32_t impl, int32_t* status, void* stream) {
-  DGPT_REQUIRE(q && k && v && o, "fmha_window: NULL pointer");
-  DGPT_REQUIRE(B >= 0 && H > 0 && Tq >= 0 && B <= 65535 && H <= 65535 && n_keys >= 0, "fmha_window: bad sizes");
-  DGPT_REQUIRE(window >= 0 && q_offset >= 0 && scale > 0.f, "fmha_window: bad window, offset or scale");
-  DGPT_REQUIRE(q_row_stride % 8 == 0 && q_batch_stride % 8 == 0 && o_row_stride % 8 == 0 && o_batch_stride % 8 == 0 &&
-                   kv_batch_stride % 8 == 0 && kv_row_stride % 8 == 0 && kv_head_stride % 8 == 0,
-               "fmha_window: strides must be multiples of 8 elements");
-  DGPT_REQUIRE(impl >= 0 && impl <= 3, "fmha_window: impl must be 0 (auto), 1 (warp-level), 2 or 3 (tensor-core)");
+// Sliding-window attention for both entry points: `kv` with keys kv_ts elements apart, dense runs or pages.
+static int fmha_sliding(const char* what, const void* q, int64_t q_batch_stride, int64_t q_row_stride, const dgpt_kv_layout& kv,
+                        int64_t kv_ts, int32_t n_keys, void* o, int64_t o_batch_stride, int64_t o_row_stride, const void* gate,
+                        int64_t gate_row_stride, int32_t B, int32_t H, int32_t G, int32_t Tq, int32_t D, int32_t q_offset,
+                        int32_t window, int32_t keep_first, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(q && o, "%s: NULL pointer", what);
+  DGPT_REQUIRE(B >= 0 && H > 0 && G > 0 && H % G == 0 && Tq >= 0 && B <= 65535 && H <= 65535 && n_keys >= 0, "%s: bad sizes", what);
+  DGPT_REQUIRE(window >= 0 && keep_first >= 0 && q_offset >= 0 && scale > 0.f, "%s: bad window, kept keys, offset or scale", what);
+  DGPT_REQUIRE(q_row_stride % 8 == 0 && q_batch_stride % 8 == 0 && o_row_stride % 8 == 0 && o_batch_stride % 8 == 0 && kv_ts > 0 &&
+                   kv_ts % 8 == 0,
+               "%s: strides must be multiples of 8 elements", what);
+  DGPT_REQUIRE(impl >= 0 && impl <= 3, "%s: impl must be 0 (auto), 1 (warp-level), 2 or 3 (tensor-core)", what);
   if (B == 0 || Tq == 0) return DGPT_OK;
-  dgpt_kv_layout kv = {};
-  kv.k_base = const_cast<void*>(k);
-  kv.v_base = const_cast<void*>(v);
-  kv.page_stride = kv_batch_stride;
-  kv.head_stride = kv_head_stride;
-  kv.page_tokens = n_keys > 0 ? n_keys : 1;
   if (int e = validate_kv(&kv, D)) return e;
+  DGPT_REQUIRE(n_keys <= (kv.page_table ? (long long)kv.max_pages * kv.page_tokens : (long long)kv.page_tokens),
+               "%s: more keys than the layout holds", what);
   FmhaArgs a;
   a.q = q; a.q_bs = q_batch_stride; a.q_rs = q_row_stride;
   a.kv_len = nullptr; a.kv_len_all = n_keys;
@@ -250,7 +251,8 @@ extern "C" int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q
   a.status = status;
   a.max_ctas = 0;
   a.pingpong = 0;
-  a.window = window; a.scale = scale; a.kv_ts = kv_row_stride;
+  a.window = window; a.scale = scale; a.kv_ts = kv_ts;
+  a.kv_heads = G; a.keep_first = keep_first;
   a.hgate = gate; a.hgate_rs = gate_row_stride;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // The persistent kernel from 1024 keys on, as for full attention, unless the window leaves a query tile only a few key
@@ -258,11 +260,36 @@ extern "C" int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q
   a.two_cta = impl == 3 || (impl == 0 && (n_keys < 1024 || (window > 0 && window <= 512)));
   const bool tc_ok = fmha_tc_supported(a, kv);
   if (impl >= 2 && !tc_ok) {
-    set_error("fmha_window: the tensor-core kernels do not cover dtype %d, head_dim %d with this layout", dtype, D);
+    set_error("%s: the tensor-core kernels do not cover dtype %d, head_dim %d with this layout", what, dtype, D);
     return DGPT_E_UNSUPPORTED;
   }
   if (tc_ok && impl != 1) return fmha_tc(a, kv, st);
   KvView view = make_view(&kv);
-  view.token_stride = kv_row_stride;
+  view.token_stride = kv_ts;
   return fmha_simt(a, view, st);
+}
+
+extern "C" int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const void* k, const void* v,
+                                int64_t kv_batch_stride, int64_t kv_row_stride, int64_t kv_head_stride, int32_t n_keys, void* o,
+                                int64_t o_batch_stride, int64_t o_row_stride, const void* gate, int64_t gate_row_stride,
+                                int32_t B, int32_t H, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, float scale,
+                                int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(kv_batch_stride % 8 == 0 && kv_head_stride % 8 == 0, "fmha_window: strides must be multiples of 8 elements");
+  dgpt_kv_layout kv = {};
+  kv.k_base = const_cast<void*>(k);
+  kv.v_base = const_cast<void*>(v);
+  kv.page_stride = kv_batch_stride;
+  kv.head_stride = kv_head_stride;
+  kv.page_tokens = n_keys > 0 ? n_keys : 1;
+  return fmha_sliding("fmha_window", q, q_batch_stride, q_row_stride, kv, kv_row_stride, n_keys, o, o_batch_stride, o_row_stride, gate,
+                      gate_row_stride, B, H, H, Tq, D, q_offset, window, 0, scale, dtype, impl, status, stream);
+}
+
+extern "C" int dgpt_fmha_grouped(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const dgpt_kv_layout* kv,
+                                 int64_t kv_token_stride, int32_t n_keys, void* o, int64_t o_batch_stride, int64_t o_row_stride,
+                                 int32_t B, int32_t H, int32_t G, int32_t Tq, int32_t D, int32_t q_offset, int32_t window,
+                                 int32_t keep_first, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(kv, "fmha_grouped: NULL pointer");
+  return fmha_sliding("fmha_grouped", q, q_batch_stride, q_row_stride, *kv, kv_token_stride, n_keys, o, o_batch_stride, o_row_stride,
+                      nullptr, 0, B, H, G, Tq, D, q_offset, window, keep_first, scale, dtype, impl, status, stream);
 }

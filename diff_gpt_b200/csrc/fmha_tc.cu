@@ -92,17 +92,18 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
   const int klen = p.kv_len ? p.kv_len[b] : p.kv_len_all;
   const int kmax = p.causal ? min(klen, p.q_offset + min(q0 + kBM, p.Tq)) : klen;
   const int tile0 = window_first_tile(p.window, p.q_offset + q0, kBN);
-  const int n_tiles = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0);
+  const int n_kept = kept_tiles(p.keep_first, tile0, kBN), kvh = h / p.kv_div;
+  const int n_tiles = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0) + n_kept;
 
   // Issue the TMA loads of key/value tile j (thread 0 only).  One box per page and per 64-wide half.
   auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t bar, int j) {
-    const int t0 = (tile0 + j) * kBN;
+    const int t0 = tile_of(j, n_kept, tile0) * kBN;
     if (pt >= kBN) {
       const int lp = t0 / pt, in = t0 - lp * pt;
       const int pg = p.page_table ? p.page_table[(long long)b * p.max_pages + lp] : b;
       mbar_expect_tx(bar, kTileBytes);
 #pragma unroll
-      for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes, map, bar, s * 64, in, h, pg);
+      for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes, map, bar, s * 64, in, kvh, pg);
     } else {
       const int per = kBN / pt;
       int valid = 0;
@@ -112,7 +113,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
         const int lp = t0 / pt + q;
         const int pg = p.page_table ? p.page_table[(long long)b * p.max_pages + lp] : b;
 #pragma unroll
-        for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes + q * pt * 128, map, bar, s * 64, 0, h, pg);
+        for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes + q * pt * 128, map, bar, s * 64, 0, kvh, pg);
       }
     }
   };
@@ -130,7 +131,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
 
   for (int j = 0; j < n_tiles; ++j) {
     const uint32_t par = (uint32_t)(j & 1);
-    const int t0 = (tile0 + j) * kBN;
+    const int t0 = tile_of(j, n_kept, tile0) * kBN;
     // ---- S = Q K^T ----
     if (tid == 0) {
       bool ok = true;
@@ -185,7 +186,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
     if (need_mask) {
 #pragma unroll
       for (int i = 0; i < kBN; ++i) {
-        sv[i] = (t0 + i <= last_key && t0 + i >= first_key) ? sv[i] : -INFINITY;
+        sv[i] = (t0 + i <= last_key && (t0 + i >= first_key || t0 + i < p.keep_first)) ? sv[i] : -INFINITY;
         mx = fmaxf(mx, sv[i]);
       }
     } else {
@@ -329,6 +330,7 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   // engine fills what lies outside the tensor with zeros - Q K^T and P V see zero columns and are unchanged
   const int d_head = a.D;
   const int D = d_head == 32 ? 64 : d_head;
+  const bool run = a.kv_ts > 0 && kv.page_table == nullptr;
   TcMaps maps;
   CUtensorMap &mq = maps.q, &mk = maps.k, &mv = maps.v;
   {
@@ -341,10 +343,10 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   {
     const int pt = kv.page_tokens;
     cuuint64_t n_pages = kv.page_table ? (kv.n_pages > 0 ? (cuuint64_t)kv.n_pages : (cuuint64_t)1 << 24) : (cuuint64_t)a.B;
-    const cuuint64_t dims[4] = {(cuuint64_t)d_head, (cuuint64_t)pt, (cuuint64_t)a.H, n_pages};
+    const cuuint64_t dims[4] = {(cuuint64_t)d_head, (cuuint64_t)pt, (cuuint64_t)(a.kv_heads > 0 ? a.kv_heads : a.H), n_pages};
     const cuuint64_t strides[3] = {(cuuint64_t)(a.kv_ts > 0 ? a.kv_ts : d_head) * 2, (cuuint64_t)kv.head_stride * 2,
                                    (cuuint64_t)kv.page_stride * 2};
-    const cuuint32_t box[4] = {64, (cuuint32_t)(pt < kBN && a.kv_ts == 0 ? pt : kBN), 1, 1};
+    const cuuint32_t box[4] = {64, (cuuint32_t)(pt < kBN && !run ? pt : kBN), 1, 1};
     if (!encode_map(&mk, kv.k_base, dims, strides, box)) return DGPT_E_CUDA;
     if (!encode_map(&mv, kv.v_base, dims, strides, box)) return DGPT_E_CUDA;
   }
@@ -353,7 +355,7 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   p.kv_len_all = a.kv_len_all;
   p.page_table = kv.page_table;
   p.max_pages = kv.max_pages;
-  p.page_tokens = a.kv_ts > 0 ? (kv.page_tokens + kBN - 1) / kBN * kBN : kv.page_tokens;  // a run is one page of whole tiles
+  p.page_tokens = run ? (kv.page_tokens + kBN - 1) / kBN * kBN : kv.page_tokens;  // a run is one page of whole tiles
   p.o = a.o;
   p.o_bs = a.o_bs;
   p.o_rs = a.o_rs;
@@ -365,6 +367,8 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   p.causal = a.causal;
   p.scale_log2 = a.scale > 0.f ? a.scale * kLog2e : kLog2e / sqrtf((float)d_head);
   p.window = a.window;
+  p.keep_first = a.window > 0 ? a.keep_first : 0;
+  p.kv_div = a.kv_heads > 0 ? a.H / a.kv_heads : 1;
   p.hgate = a.hgate;
   p.hgate_rs = a.hgate_rs;
   p.d_head = d_head;

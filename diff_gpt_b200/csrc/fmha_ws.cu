@@ -35,7 +35,7 @@ constexpr int kWsThreads = 320;  // 8 softmax warps, the MMA issuer's warp, the 
 constexpr uint32_t kWsTmemCols = 512;
 
 struct WsItem {
-  int b, h, q0, klen, tile0, n;  // n = key tiles, the first of them tile0 (0 unless a sliding window cuts the rest off)
+  int b, h, q0, klen, tile0, n_kept, n;  // n = key tiles: n_kept of kept first keys, then those from tile0 on (see tile_of)
 };
 
 __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
@@ -46,7 +46,8 @@ __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
   it.klen = p.kv_len ? p.kv_len[it.b] : p.kv_len_all;
   const int kmax = p.causal ? min(it.klen, p.q_offset + min(it.q0 + kBM, p.Tq)) : it.klen;
   it.tile0 = window_first_tile(p.window, p.q_offset + it.q0, kBN);
-  it.n = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0);
+  it.n_kept = kept_tiles(p.keep_first, it.tile0, kBN);
+  it.n = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0) + it.n_kept;
   return it;
 }
 
@@ -119,13 +120,13 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         const WsItem it = ws_item(p, bh, qt);
         if (it.n == 0) continue;
         auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t full, int j) {
-          const int t0 = (it.tile0 + j) * kBN;
+          const int t0 = tile_of(j, it.n_kept, it.tile0) * kBN, kvh = it.h / p.kv_div;
           if (pt >= kBN) {
             const int lp = t0 / pt, in = t0 - lp * pt;
             const int pg = p.page_table ? p.page_table[(long long)it.b * p.max_pages + lp] : it.b;
             mbar_expect_tx(full, kTileBytes);
 #pragma unroll
-            for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes, map, full, s * 64, in, it.h, pg);
+            for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes, map, full, s * 64, in, kvh, pg);
           } else {
             const int per = kBN / pt;
             int valid = 0;
@@ -135,7 +136,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
               const int lp = t0 / pt + q;
               const int pg = p.page_table ? p.page_table[(long long)it.b * p.max_pages + lp] : it.b;
 #pragma unroll
-              for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes + q * pt * 128, map, full, s * 64, 0, it.h, pg);
+              for (int s = 0; s < kSub; ++s) tma_load_4d(dst + s * kSubBytes + q * pt * 128, map, full, s * 64, 0, kvh, pg);
             }
           }
         };
@@ -265,7 +266,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       float m = -INFINITY, l = 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const unsigned g = g0 + (unsigned)j, buf = g & 1u, ph = (g >> 1) & 1u;
-        const int t0 = (it.tile0 + j) * kBN;
+        const int t0 = tile_of(j, it.n_kept, it.tile0) * kBN;
         // exits are taken by whole warps (the vote makes the decision uniform), never by single lanes
         if (!__all_sync(0xffffffffu, wait_or_abort(bar_s0 + 8 * buf, ph, abort_flag, 23))) {
           fail = true;
@@ -299,7 +300,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         tc_wait_ld();
         if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key && c0 + i >= first_key) ? sv[i] : -INFINITY;
+          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key && (c0 + i >= first_key || c0 + i < p.keep_first)) ? sv[i] : -INFINITY;
         }
         // One sweep turns this thread's 64 scores into probabilities against a reference maximum `ref` (log2 domain),
         // writes them as packed bf16 into the P buffer and returns their sum.

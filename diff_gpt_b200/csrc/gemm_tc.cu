@@ -6,6 +6,7 @@
 //   mode 1:  out[m, n / 2] = swiglu(bf16(acc[m, n]), bf16(acc[m, n + 1]))   for even n  (interleaved gate / linear)
 //   mode 2:  out[m, n]     = bf16(resid[m, n] + acc[m, n])                    (the residual add of addmm, one rounding)
 //   mode 4:  out[m, n]     = bf16(xielu(acc[m, n]))   with alpha_p = alpha, alpha_n = limit
+//   mode 5:  out[m, n / 2] = bf16(silu(acc[m, n]) * acc[m, n + 1])   for even n  (interleaved gate / up)
 //   mode 3:  nothing is stored: row m keeps the best key of  key[m, n] = cap(bf16(acc[m, n])) / T + Gumbel noise(m, n)
 //            (no noise and T = 1 for an arg-max) in best[m], a 64-bit word (order-preserving key bits, ~n) raised with
 //            atomicMax - the tied-embedding head with the draw in its epilogue, so [M, N] logits never reach HBM
@@ -225,7 +226,7 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ C
           continue;
         }
         if (DRAW) continue;
-        if (p.mode != 1) {
+        if (p.mode != 1 && p.mode != 5) {
           __nv_bfloat16* dst = p.out + (long long)row * p.out_rs + col0 + c;
 #pragma unroll
           for (int q = 0; q < 4; ++q) {
@@ -244,6 +245,10 @@ gemm_tc_kernel(const __grid_constant__ CUtensorMap ma, const __grid_constant__ C
         } else {
           using B = Io<__nv_bfloat16>;
           float r[16];
+          if (p.mode == 5) {
+#pragma unroll
+            for (int k = 0; k < 16; ++k) r[k] = silu_mul_fast(v[2 * k], v[2 * k + 1]);
+          } else
 #pragma unroll
           for (int k = 0; k < 16; ++k) {
             // the reference's Linear writes bf16 before the activation reads it
@@ -334,8 +339,8 @@ int dgpt::linear_launch(const void* a, int64_t a_row_stride, const void* w, int6
                         const HeadDraw* draw, void* stream) {
   DGPT_REQUIRE(a && w && (out || epilogue == 3), "linear: NULL pointer");
   DGPT_REQUIRE(M >= 0 && N > 0 && K > 0, "linear: bad sizes");
-  DGPT_REQUIRE(epilogue >= 0 && epilogue <= 4,
-               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add), 3 (draw) or 4 (xIELU)");
+  DGPT_REQUIRE(epilogue >= 0 && epilogue <= 5,
+               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add), 3 (draw), 4 (xIELU) or 5 (SiLU gate)");
   DGPT_REQUIRE(epilogue != 2 || resid, "linear: epilogue 2 needs the matrix to add");
   DGPT_REQUIRE(epilogue != 3 || (draw && draw->best), "linear: epilogue 3 needs the draw parameters");
   if (dtype != DGPT_BF16) {
@@ -418,8 +423,8 @@ extern "C" int dgpt_linear(const void* a, int64_t a_row_stride, const void* w, i
                            int64_t out_row_stride, const void* resid, int64_t resid_row_stride, int32_t M, int32_t N,
                            int32_t K, int32_t epilogue, float alpha, float limit, int32_t dtype, int32_t* status,
                            void* stream) {
-  DGPT_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 4,
-               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add) or 4 (xIELU)");
+  DGPT_REQUIRE((epilogue >= 0 && epilogue <= 2) || epilogue == 4 || epilogue == 5,
+               "linear: epilogue must be 0 (store), 1 (SwiGLU of interleaved pairs), 2 (add), 4 (xIELU) or 5 (SiLU gate)");
   return linear_launch(a, a_row_stride, w, w_row_stride, out, out_row_stride, resid, resid_row_stride, M, N, K, epilogue, alpha,
                        limit, dtype, status, nullptr, stream);
 }

@@ -1,7 +1,10 @@
-// Attention over a cache of latents (one vector of r numbers per token, shared by all heads) with the key and value
-// expansions absorbed into the query and the output: q~_h = W_uk,h^T q_h and o_h = W_uv,h (sum_j p_j c_j), so scores and
-// sums are formed on the latents themselves and the cache is read once for all heads.  A sliding window limits which
-// latents a query sees.
+// Attention over cached rows, few queries per sequence (decoding, short portions), with a sliding window and a number of
+// first tokens that stay visible.  Two kinds of row (see latent_attn.cuh):
+//   latents       one vector of r numbers per token, shared by all heads, with the key and value expansions absorbed into
+//                 the query and the output: q~_h = W_uk,h^T q_h and o_h = W_uv,h (sum_j p_j c_j), so scores and sums are
+//                 formed on the latents themselves
+//   keys, values  of G groups of heads (grouped-query attention)
+// Either way a cached row is read once for all heads that share it.
 //
 //   latent_append_kernel   c = rms_norm(x) * w, rounded once, into the paged cache (and a flat copy where asked for)
 //   latent_tc_kernel       latent_tc.cu: bf16 on tcgen05, the form that serves
@@ -13,7 +16,7 @@ namespace dgpt {
 
 constexpr int kLatThreads = 256;
 
-// this split's part [begin, end) of a row's keys
+// this split's part [begin, end) of the keys a row sees, counted along [0, ks) and then [lo, n)
 struct LatentSpan {
   LatentKeys k;
   int begin, end;
@@ -21,13 +24,15 @@ struct LatentSpan {
 __device__ __forceinline__ LatentSpan latent_span(const LatentArgs& a, int row, int split) {
   LatentSpan sp;
   sp.k = latent_keys(a, row);
-  const int chunk = (sp.k.n - sp.k.lo + a.n_splits - 1) / a.n_splits;
-  sp.begin = min(sp.k.n, sp.k.lo + split * chunk);
-  sp.end = min(sp.k.n, sp.begin + chunk);
+  const int seen = sp.k.ks + sp.k.n - sp.k.lo;
+  const int chunk = (seen + a.n_splits - 1) / a.n_splits;
+  sp.begin = min(seen, split * chunk);
+  sp.end = min(seen, sp.begin + chunk);
   return sp;
 }
-// Element offset of logical key i, or -1 when its table entry lies outside the pool (such a latent counts as zeros).
-__device__ __forceinline__ long long latent_offset(const LatentArgs& a, const LatentKeys& k, int i) {
+// Element offset of the cache row of seen key j, or -1 when its table entry lies outside the pool (such a row counts as zeros).
+__device__ __forceinline__ long long latent_offset(const LatentArgs& a, const LatentKeys& k, int j) {
+  const int i = j < k.ks ? j : k.lo + (j - k.ks);
   const int slot = i < k.n0 ? i : k.s1 + (i - k.n0);
   const int lp = slot / a.kv.page_tokens;
   const int in = slot - lp * a.kv.page_tokens;
@@ -36,7 +41,7 @@ __device__ __forceinline__ long long latent_offset(const LatentArgs& a, const La
     pg = a.kv.page_table[(long long)k.seq * a.kv.max_pages + lp];
     if (a.kv.n_pages > 0 && (pg < 0 || pg >= a.kv.n_pages)) return -1;
   }
-  return pg * a.kv.page_stride + (long long)in * a.r;
+  return pg * a.kv.page_stride + (long long)in * a.row_w;
 }
 
 // ---- append: one warp per token ---------------------------------------------------------------
@@ -106,26 +111,29 @@ __global__ void latent_append_kernel(const T* __restrict__ in, long long in_rs, 
   }
 }
 
-// ---- any r, any storage type, CUDA cores -------------------------------------------------------
-// Shared memory: q and o of `hg` heads in fp32, a tile of `tt` latents in fp32 (row stride r + 1), scores.
+// ---- any sizes, any storage type, CUDA cores ------------------------------------------------------
+// Shared memory: q and o of `hg` heads of one group in fp32, a tile of `tt` keys (row stride dk + 1) and of their values
+// (dv + 1; the same tile where the values are the keys), scores.
 template <typename T>
 __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(const LatentArgs a, int hg, int tt) {
   extern __shared__ __align__(16) uint8_t lat_raw[];
-  const int r = a.r, ldc = r + 1;
-  float* sq = reinterpret_cast<float*>(lat_raw);  // [hg][r]
-  float* so = sq + hg * r;                        // [hg][r]
-  float* sc = so + hg * r;                        // [tt][r + 1]
-  float* sp_ = sc + tt * ldc;                     // [hg][tt]
+  const int dk = a.dk, dv = a.dv, ldk = dk + 1, ldv = dv + 1;
+  const bool same = a.v_col == 0;
+  float* sq = reinterpret_cast<float*>(lat_raw);  // [hg][dk]
+  float* so = sq + hg * dk;                       // [hg][dv]
+  float* sk = so + hg * dv;                       // [tt][dk + 1]
+  float* sv = same ? sk : sk + tt * ldk;          // [tt][dv + 1]
+  float* sp_ = sv + tt * ldv;                     // [hg][tt]
   float* sm = sp_ + hg * tt;                      // [hg] running maximum, [hg] sum, [hg] rescale
   const int tid = threadIdx.x;
-  const int row = blockIdx.x, split = blockIdx.y, h0 = blockIdx.z * hg;
-  const int nh = min(hg, a.H - h0);
+  const int row = blockIdx.x, split = blockIdx.y;
+  const int per = a.H / a.G, n_hg = (per + hg - 1) / hg;
+  const int g = blockIdx.z / n_hg, hi = (blockIdx.z - g * n_hg) * hg;
+  const int h0 = g * per + hi, nh = min(hg, per - hi);
   const LatentSpan sp = latent_span(a, row, split);
-  const T* q = static_cast<const T*>(a.q) + (long long)row * a.q_rs + (long long)h0 * r;
-  for (int i = tid; i < nh * r; i += kLatThreads) {
-    sq[i] = Io<T>::ld(q + i) * a.scale_log2;
-    so[i] = 0.f;
-  }
+  const T* q = static_cast<const T*>(a.q) + (long long)row * a.q_rs + (long long)h0 * dk;
+  for (int i = tid; i < nh * dk; i += kLatThreads) sq[i] = Io<T>::ld(q + i) * a.scale_log2;
+  for (int i = tid; i < nh * dv; i += kLatThreads) so[i] = 0.f;
   if (tid < nh) {
     sm[tid] = -INFINITY;
     sm[hg + tid] = 0.f;
@@ -136,22 +144,27 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(const LatentAr
     __syncthreads();
     for (int t = tid >> 5; t < cnt; t += kLatThreads / 32) {
       const long long off = latent_offset(a, sp.k, i0 + t);
-      for (int c = tid & 31; c < r; c += 32) sc[t * ldc + c] = off < 0 ? 0.f : Io<T>::ld(pool + off + c);
+      const T* src = pool + off + g * dk;
+      for (int c = tid & 31; c < dk; c += 32) sk[t * ldk + c] = off < 0 ? 0.f : Io<T>::ld(src + c);
+      if (!same) {
+        src = pool + off + a.v_col + g * dv;
+        for (int c = tid & 31; c < dv; c += 32) sv[t * ldv + c] = off < 0 ? 0.f : Io<T>::ld(src + c);
+      }
     }
     __syncthreads();
     for (int i = tid; i < nh * cnt; i += kLatThreads) {
       const int h = i / cnt, t = i - h * cnt;
-      const float* qh = sq + h * r;
-      const float* ct = sc + t * ldc;
+      const float* qh = sq + h * dk;
+      const float* ct = sk + t * ldk;
       float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
       int c = 0;
-      for (; c + 4 <= r; c += 4) {
+      for (; c + 4 <= dk; c += 4) {
         d0 += qh[c] * ct[c];
         d1 += qh[c + 1] * ct[c + 1];
         d2 += qh[c + 2] * ct[c + 2];
         d3 += qh[c + 3] * ct[c + 3];
       }
-      for (; c < r; ++c) d0 += qh[c] * ct[c];
+      for (; c < dk; ++c) d0 += qh[c] * ct[c];
       sp_[h * tt + t] = (d0 + d1) + (d2 + d3);
     }
     __syncthreads();
@@ -176,22 +189,22 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(const LatentAr
       }
     }
     __syncthreads();
-    for (int i = tid; i < nh * r; i += kLatThreads) {
-      const int h = i / r, c = i - h * r;
+    for (int i = tid; i < nh * dv; i += kLatThreads) {
+      const int h = i / dv, c = i - h * dv;
       float acc = so[i] * sm[2 * hg + h];
-      for (int t = 0; t < cnt; ++t) acc += sp_[h * tt + t] * sc[t * ldc + c];
+      for (int t = 0; t < cnt; ++t) acc += sp_[h * tt + t] * sv[t * ldv + c];
       so[i] = acc;
     }
   }
   __syncthreads();
   const long long RH = (long long)a.n_seq * a.Tn * a.H;
-  for (int i = tid; i < nh * r; i += kLatThreads) {
-    const int h = i / r, c = i - h * r;
+  for (int i = tid; i < nh * dv; i += kLatThreads) {
+    const int h = i / dv, c = i - h * dv;
     const long long rh = (long long)row * a.H + h0 + h;
     const float sum = sm[hg + h];
     if (a.n_splits > 1) {
       const long long slot = (long long)split * RH + rh;
-      a.ws_o[slot * r + c] = so[i];
+      a.ws_o[slot * dv + c] = so[i];
       if (c == 0) {
         a.ws_ml[2 * slot] = sm[h];
         a.ws_ml[2 * slot + 1] = sum;
@@ -199,7 +212,7 @@ __global__ void __launch_bounds__(kLatThreads) latent_attn_kernel(const LatentAr
     } else {
       float f = sum > 0.f ? 1.f / sum : 0.f;
       if (a.gate) f *= 1.f / (1.f + expf(-Io<T>::ld(static_cast<const T*>(a.gate) + (long long)row * a.gate_rs + h0 + h)));
-      Io<T>::st(static_cast<T*>(a.out) + (long long)row * a.out_rs + (long long)(h0 + h) * r + c, so[i] * f);
+      Io<T>::st(static_cast<T*>(a.out) + (long long)row * a.out_rs + (long long)(h0 + h) * dv + c, so[i] * f);
     }
   }
 }
@@ -227,18 +240,18 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const LatentArgs a)
   l = block_sum(l, scratch);  // and `wt` is complete
   float f = l > 0.f ? 1.f / l : 0.f;
   if (a.gate) f *= 1.f / (1.f + expf(-Io<T>::ld(static_cast<const T*>(a.gate) + row * a.gate_rs + h)));
-  T* dst = static_cast<T*>(a.out) + row * a.out_rs + (long long)h * a.r;
-  for (int c = tid; c < a.r; c += 128) {
+  T* dst = static_cast<T*>(a.out) + row * a.out_rs + (long long)h * a.dv;
+  for (int c = tid; c < a.dv; c += 128) {
     float acc = 0.f;
     int s = 0;
     for (; s + 8 <= n; s += 8) {  // eight loads in flight; a split without keys has weight 0 and holds nothing
       float v[8];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) v[u] = a.ws_o[((s + u) * RH + rh) * a.r + c];
+      for (int u = 0; u < 8; ++u) v[u] = a.ws_o[((s + u) * RH + rh) * a.dv + c];
 #pragma unroll
       for (int u = 0; u < 8; ++u) acc += wt[s + u] == 0.f ? 0.f : wt[s + u] * v[u];
     }
-    for (; s < n; ++s) acc += wt[s] == 0.f ? 0.f : wt[s] * a.ws_o[(s * RH + rh) * a.r + c];
+    for (; s < n; ++s) acc += wt[s] == 0.f ? 0.f : wt[s] * a.ws_o[(s * RH + rh) * a.dv + c];
     Io<T>::st(dst + c, acc * f);
   }
 }
@@ -254,15 +267,18 @@ static int latent_max_smem() {
 template <typename T>
 static int latent_simt_launch(const LatentArgs& a, cudaStream_t st) {
   const int limit = latent_max_smem();
-  auto need = [&](int hg, int tt) { return ((size_t)2 * hg * a.r + (size_t)tt * (a.r + 1) + (size_t)hg * tt + 3 * hg) * 4; };
-  int hg = a.H < 16 ? a.H : 16, tt = 32;
+  const int per = a.H / a.G;
+  auto need = [&](int hg, int tt) {
+    return ((size_t)hg * (a.dk + a.dv) + (size_t)tt * (a.dk + 1 + (a.v_col ? a.dv + 1 : 0)) + (size_t)hg * tt + 3 * hg) * 4;
+  };
+  int hg = per < 16 ? per : 16, tt = 32;
   while (need(hg, tt) > (size_t)limit && (hg > 1 || tt > 1)) {
     if (hg > 4 || (tt == 1 && hg > 1)) hg = (hg + 1) / 2;
     else tt = tt / 2;
   }
   const size_t smem = need(hg, tt);
   if (smem > (size_t)limit) {
-    set_error("latent_attn: r = %d does not fit the shared memory", a.r);
+    set_error("latent_attn: key size %d and value size %d do not fit the shared memory", a.dk, a.dv);
     return DGPT_E_UNSUPPORTED;
   }
   cudaError_t e = cudaFuncSetAttribute(latent_attn_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -270,7 +286,7 @@ static int latent_simt_launch(const LatentArgs& a, cudaStream_t st) {
     set_error("latent_attn: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     return DGPT_E_CUDA;
   }
-  const dim3 grid((unsigned)(a.n_seq * a.Tn), (unsigned)a.n_splits, (unsigned)((a.H + hg - 1) / hg));
+  const dim3 grid((unsigned)(a.n_seq * a.Tn), (unsigned)a.n_splits, (unsigned)(a.G * ((per + hg - 1) / hg)));
   latent_attn_kernel<T><<<grid, kLatThreads, smem, st>>>(a, hg, tt);
   return launch_status("latent_attn");
 }
@@ -318,27 +334,31 @@ extern "C" size_t dgpt_latent_attn_workspace_bytes(int32_t R, int32_t H, int32_t
   return (((size_t)R * H * n_splits * (size_t)(r + 2) * sizeof(float)) + 15) & ~(size_t)15;
 }
 
-extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, const int32_t* len0,
-                                const int32_t* start1, const int32_t* len1, const int32_t* step_ptr, const void* gate,
-                                int64_t gate_row_stride, void* out, int64_t out_row_stride, void* workspace,
-                                size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T, int32_t H, int32_t r,
-                                int32_t window, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
-  DGPT_REQUIRE(q && out && start1 && len1, "latent_attn: NULL pointer");
-  DGPT_REQUIRE(n_seq >= 0 && T >= 0 && H > 0 && r > 0 && r % 8 == 0 && window >= 0, "latent_attn: bad sizes");
-  DGPT_REQUIRE(n_splits >= 1 && n_splits <= kLatMaxSplits && H <= 65535,
-               "latent_attn: 1 to %d splits", kLatMaxSplits);
-  DGPT_REQUIRE(impl >= 0 && impl <= 2, "latent_attn: impl must be 0 (auto), 1 (CUDA cores) or 2 (tcgen05)");
-  DGPT_REQUIRE(dtype == DGPT_F32 || dtype == DGPT_BF16, "latent_attn: unknown dtype %d", dtype);
+// Checks, the choice of kernel and the merge of splits for both entry points.
+static int row_attn(const char* what, const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, int32_t row_w, int32_t v_col,
+                    const int32_t* len0, const int32_t* start1, const int32_t* len1, const int32_t* step_ptr, const void* gate,
+                    int64_t gate_row_stride, void* out, int64_t out_row_stride, void* workspace, size_t workspace_bytes,
+                    int32_t n_splits, int32_t n_seq, int32_t T, int32_t H, int32_t G, int32_t dk, int32_t dv, int32_t window,
+                    int32_t keep_first, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(q && out && start1 && len1, "%s: NULL pointer", what);
+  DGPT_REQUIRE(n_seq >= 0 && T >= 0 && H > 0 && G > 0 && H % G == 0 && dk > 0 && dk % 8 == 0 && dv > 0 && dv % 8 == 0 && window >= 0 &&
+                   keep_first >= 0,
+               "%s: bad sizes", what);
+  DGPT_REQUIRE(row_w % 8 == 0 && v_col % 8 == 0 && row_w >= G * dk && (v_col == 0 ? dk == dv && G == 1 : v_col >= G * dk && row_w >= v_col + G * dv),
+               "%s: keys and values do not fit a cache row of %d", what, row_w);
+  DGPT_REQUIRE(n_splits >= 1 && n_splits <= kLatMaxSplits && H <= 65535, "%s: 1 to %d splits", what, kLatMaxSplits);
+  DGPT_REQUIRE(impl >= 0 && impl <= 2, "%s: impl must be 0 (auto), 1 (CUDA cores) or 2 (tcgen05)", what);
+  DGPT_REQUIRE(dtype == DGPT_F32 || dtype == DGPT_BF16, "%s: unknown dtype %d", what, dtype);
   DGPT_REQUIRE((reinterpret_cast<uintptr_t>(q) & 15) == 0 && q_row_stride % 8 == 0 && (reinterpret_cast<uintptr_t>(out) & 15) == 0 &&
                    out_row_stride % 8 == 0,
-               "latent_attn: q and out must be 16-byte aligned with row strides of a multiple of 8");
-  if (int e = validate_kv(kv, r)) return e;
+               "%s: q and out must be 16-byte aligned with row strides of a multiple of 8", what);
+  if (int e = validate_kv(kv, row_w)) return e;
   const long long R = (long long)n_seq * T;
   if (R == 0) return DGPT_OK;
-  DGPT_REQUIRE(R <= 0x7fffffff, "latent_attn: too many rows");
-  const size_t need = dgpt_latent_attn_workspace_bytes((int32_t)R, H, r, n_splits);
+  DGPT_REQUIRE(R <= 0x7fffffff, "%s: too many rows", what);
+  const size_t need = dgpt_latent_attn_workspace_bytes((int32_t)R, H, dv, n_splits);
   if (need > 0 && (workspace == nullptr || workspace_bytes < need || (reinterpret_cast<uintptr_t>(workspace) & 15) != 0)) {
-    set_error("latent_attn: a 16-byte aligned workspace of %zu bytes is needed, %zu given", need, workspace_bytes);
+    set_error("%s: a 16-byte aligned workspace of %zu bytes is needed, %zu given", what, need, workspace_bytes);
     return DGPT_E_WORKSPACE;
   }
   LatentArgs a;
@@ -348,15 +368,16 @@ extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_
   a.gate = gate; a.gate_rs = gate_row_stride;
   a.out = out; a.out_rs = out_row_stride;
   a.ws_o = static_cast<float*>(workspace);
-  a.ws_ml = workspace ? a.ws_o + (size_t)R * H * n_splits * r : nullptr;
-  a.n_splits = n_splits; a.n_seq = n_seq; a.Tn = T; a.H = H; a.r = r; a.window = window;
+  a.ws_ml = workspace ? a.ws_o + (size_t)R * H * n_splits * dv : nullptr;
+  a.n_splits = n_splits; a.n_seq = n_seq; a.Tn = T; a.H = H; a.window = window;
+  a.G = G; a.dk = dk; a.dv = dv; a.row_w = row_w; a.v_col = v_col; a.keep = keep_first;
   a.scale_log2 = scale * kLog2e;
   a.status = status;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const bool tc_ok = latent_tc_supported(a, *kv, dtype);
   if (impl == 2 && !tc_ok) {
-    set_error("latent_attn: the tcgen05 kernel covers bf16 with r <= 512 in dense runs or pages that tile 128 keys (r = %d, dtype %d, "
-              "page_tokens %d)", r, dtype, kv->page_tokens);
+    set_error("%s: the tcgen05 kernel covers bf16 with key and value sizes up to 512 in dense runs or pages that tile 128 keys "
+              "(sizes %d and %d, dtype %d, page_tokens %d)", what, dk, dv, dtype, kv->page_tokens);
     return DGPT_E_UNSUPPORTED;
   }
   int e;
@@ -368,4 +389,25 @@ extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_
   if (dtype == DGPT_F32) latent_combine_kernel<float><<<(unsigned)RH, 128, 0, st>>>(a);
   else latent_combine_kernel<__nv_bfloat16><<<(unsigned)RH, 128, 0, st>>>(a);
   return launch_status("latent_combine");
+}
+
+extern "C" int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, const int32_t* len0,
+                                const int32_t* start1, const int32_t* len1, const int32_t* step_ptr, const void* gate,
+                                int64_t gate_row_stride, void* out, int64_t out_row_stride, void* workspace,
+                                size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T, int32_t H, int32_t r,
+                                int32_t window, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
+  return row_attn("latent_attn", q, q_row_stride, kv, r, 0, len0, start1, len1, step_ptr, gate, gate_row_stride, out, out_row_stride,
+                  workspace, workspace_bytes, n_splits, n_seq, T, H, 1, r, r, window, 0, scale, dtype, impl, status, stream);
+}
+
+extern "C" int dgpt_grouped_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, int32_t row_width, int32_t v_col,
+                                 const int32_t* len0, const int32_t* start1, const int32_t* len1, const int32_t* step_ptr,
+                                 const void* gate, int64_t gate_row_stride, void* out, int64_t out_row_stride, void* workspace,
+                                 size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T, int32_t H, int32_t G,
+                                 int32_t dk, int32_t dv, int32_t window, int32_t keep_first, float scale, int32_t dtype,
+                                 int32_t impl, int32_t* status, void* stream) {
+  DGPT_REQUIRE(v_col > 0, "grouped_attn: the values follow the keys in a cache row");
+  return row_attn("grouped_attn", q, q_row_stride, kv, row_width, v_col, len0, start1, len1, step_ptr, gate, gate_row_stride, out,
+                  out_row_stride, workspace, workspace_bytes, n_splits, n_seq, T, H, G, dk, dv, window, keep_first, scale, dtype, impl,
+                  status, stream);
 }

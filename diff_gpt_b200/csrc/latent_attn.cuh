@@ -1,4 +1,8 @@
-// Arguments and key ranges shared by the latent-attention kernels (latent_attn.cu, latent_tc.cu).
+// Arguments and key ranges shared by the kernels that attend to cached rows (latent_attn.cu, latent_tc.cu).
+//
+// A cache holds one row of `row_w` numbers per token.  Query head h belongs to group g = h / (H / G); the group's key is
+// columns [g dk, +dk) of a row and its value columns [v_col + g dv, +dv).  Attention on latents is the case of one group
+// whose value is its key (dk = dv, v_col = 0); grouped-query attention stores the G keys and then the G values.
 #pragma once
 
 #include "common.cuh"
@@ -19,14 +23,17 @@ struct LatentArgs {
   long long out_rs;
   float* ws_o;
   float* ws_ml;
-  int n_splits, n_seq, Tn, H, r, window;
+  int n_splits, n_seq, Tn, H, window;
+  int G, dk, dv;    // groups, query / key size, value size
+  int row_w, v_col; // elements between rows; where the values start
+  int keep;         // the first `keep` keys are seen from every distance
   float scale_log2;
   int* status;
 };
 
-// The keys of one row: logical keys [lo, n); key i is slot i below n0 and slot s1 + (i - n0) from there on.
+// The keys of one query row: logical keys [0, ks) and [lo, n); key i is slot i below n0 and slot s1 + (i - n0) from there on.
 struct LatentKeys {
-  int seq, n0, s1, lo, n;
+  int seq, n0, s1, ks, lo, n;
 };
 __device__ __forceinline__ LatentKeys latent_keys(const LatentArgs& a, int row) {
   LatentKeys k;
@@ -38,10 +45,11 @@ __device__ __forceinline__ LatentKeys latent_keys(const LatentArgs& a, int row) 
   const int n1 = a.len1[k.seq] + (a.step_ptr ? *a.step_ptr : 0) + t;
   k.n = k.n0 + min(max(n1, 0), cap - k.s1);  // never past the sequence's slots
   k.lo = a.window > 0 ? max(0, k.n - a.window) : 0;
+  k.ks = min(a.keep, k.lo);
   return k;
 }
 
-// tcgen05 form (latent_tc.cu): bf16, r <= 512, dense runs or pages that tile its 128-key blocks
+// tcgen05 form (latent_tc.cu): bf16, dk, dv <= 512, dense runs or pages that tile its 128-key blocks
 bool latent_tc_supported(const LatentArgs& a, const dgpt_kv_layout& kv, int dtype);
 int latent_tc_launch(const LatentArgs& a, const dgpt_kv_layout& kv, cudaStream_t st);
 

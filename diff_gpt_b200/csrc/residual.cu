@@ -5,66 +5,17 @@
 //   depth_avg_conv   x = sum_j a_j X_j ;  h = x + causal_conv(x)      (h is what the next mixer reads)
 //   layer_tail       the two above in one pass for one new token per sequence (decode)
 //   depth_avg_norm   x = sum_j a_j X_j ;  out = rms_norm(x) * w        (in front of the output head)
-//   xielu            the activation, element-wise (the GEMM of gemm_tc.cu has it as an epilogue)
+//   xielu, silu_mul  activations, element-wise (the GEMM of gemm_tc.cu has them as epilogues)
 //
 // X_j are the fp32 [n, C] slices of one slab, `term_stride` elements apart; everything is accumulated in fp32.
 // All of them are HBM-bound: each X_j row is read once and each output row written once.  VEC = 4 channels per thread
 // where C is a multiple of 4, 1 otherwise.
 #include "activation.cuh"
-#include "common.cuh"
+#include "rowvec.cuh"
 
 namespace dgpt {
 
-constexpr int kRowThreads = 256;
 constexpr int kMaxTaps = 16;
-
-template <int VEC>
-struct FVec {
-  float v[VEC];
-};
-
-template <int VEC>
-__device__ __forceinline__ FVec<VEC> ldf(const float* p) {
-  FVec<VEC> r;
-  if constexpr (VEC == 4) {
-    const float4 t = *reinterpret_cast<const float4*>(p);
-    r.v[0] = t.x; r.v[1] = t.y; r.v[2] = t.z; r.v[3] = t.w;
-  } else {
-    r.v[0] = *p;
-  }
-  return r;
-}
-template <int VEC>
-__device__ __forceinline__ void stf(float* p, const FVec<VEC>& r) {
-  if constexpr (VEC == 4) *reinterpret_cast<float4*>(p) = make_float4(r.v[0], r.v[1], r.v[2], r.v[3]);
-  else *p = r.v[0];
-}
-// VEC values of storage type T
-template <typename T, int VEC>
-__device__ __forceinline__ FVec<VEC> ldt(const T* p) {
-  FVec<VEC> r;
-  if constexpr (VEC == 1) {
-    r.v[0] = Io<T>::ld(p);
-  } else if constexpr (sizeof(T) == 4) {
-    return ldf<VEC>(reinterpret_cast<const float*>(p));
-  } else {
-    const uint2 t = *reinterpret_cast<const uint2*>(p);
-    r.v[0] = __uint_as_float(t.x << 16); r.v[1] = __uint_as_float(t.x & 0xffff0000u);
-    r.v[2] = __uint_as_float(t.y << 16); r.v[3] = __uint_as_float(t.y & 0xffff0000u);
-  }
-  return r;
-}
-template <typename T, int VEC>
-__device__ __forceinline__ void stt(T* p, const FVec<VEC>& r) {
-  if constexpr (VEC == 1) {
-    Io<T>::st(p, r.v[0]);
-  } else if constexpr (sizeof(T) == 4) {
-    stf<VEC>(reinterpret_cast<float*>(p), r);
-  } else {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(r.v[0], r.v[1]), b = __floats2bfloat162_rn(r.v[2], r.v[3]);
-    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
-  }
-}
 
 // sum_j coef[j] * slab[j][off .. off + VEC)
 template <int VEC>
@@ -312,10 +263,24 @@ __global__ void xielu_kernel(const T* __restrict__ in, T* __restrict__ out, long
   stt<T, VEC>(out + i, t);
 }
 
-static bool al16(const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; }
-
-// Row kernels: threads per CTA and vectors per thread for a row of `cv` vectors
-static int row_threads(int cv) { return cv >= 256 ? 256 : (cv > 64 ? (cv + 31) / 32 * 32 : 64); }
+// out[i] = silu(in[2 i]) * in[2 i + 1]: gate and up columns interleaved
+template <typename T, int VEC>
+__global__ void silu_mul_kernel(const T* __restrict__ in, T* __restrict__ out, long long n_out) {
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * VEC;
+  if (i >= n_out) return;
+  FVec<VEC> a, b, r;
+  if constexpr (VEC == 4) {
+    a = ldt<T, VEC>(in + 2 * i);
+    b = ldt<T, VEC>(in + 2 * i + 4);
+    r.v[0] = silu_mul_value(a.v[0], a.v[1]);
+    r.v[1] = silu_mul_value(a.v[2], a.v[3]);
+    r.v[2] = silu_mul_value(b.v[0], b.v[1]);
+    r.v[3] = silu_mul_value(b.v[2], b.v[3]);
+  } else {
+    r.v[0] = silu_mul_value(Io<T>::ld(in + 2 * i), Io<T>::ld(in + 2 * i + 1));
+  }
+  stt<T, VEC>(out + i, r);
+}
 
 }  // namespace dgpt
 
@@ -493,4 +458,24 @@ extern "C" int dgpt_xielu(const void* in, void* out, int64_t n, float alpha_p, f
   }
 #undef DGPT_XI
   return launch_status("xielu");
+}
+
+extern "C" int dgpt_silu_mul(const void* in, void* out, int64_t n_out, int32_t dtype, void* stream) {
+  DGPT_REQUIRE(in && out && n_out >= 0, "silu_mul: bad arguments");
+  DGPT_REQUIRE(dtype == DGPT_F32 || dtype == DGPT_BF16, "silu_mul: unknown dtype %d", dtype);
+  if (n_out == 0) return DGPT_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool v4 = n_out % 4 == 0 && al16(in) && al16(out);
+  const long long work = v4 ? n_out / 4 : n_out;
+  const unsigned grid = (unsigned)((work + 255) / 256);
+#define DGPT_SM(TT, VV) silu_mul_kernel<TT, VV><<<grid, 256, 0, st>>>(static_cast<const TT*>(in), static_cast<TT*>(out), n_out)
+  if (dtype == DGPT_F32) {
+    if (v4) DGPT_SM(float, 4);
+    else DGPT_SM(float, 1);
+  } else {
+    if (v4) DGPT_SM(__nv_bfloat16, 4);
+    else DGPT_SM(__nv_bfloat16, 1);
+  }
+#undef DGPT_SM
+  return launch_status("silu_mul");
 }

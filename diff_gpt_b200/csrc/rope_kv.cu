@@ -169,6 +169,96 @@ static int rope_vec_launch(const void* q, const void* k, const void* v, long lon
   return launch_status("rope_qknorm_kvappend");
 }
 
+// ---- norm over whole projections, rotation of the leading dimensions, append to a cache of rows ------------------
+// CTA per token.  q and k are normalised over all their heads at once, then the first `rot` dimensions of each head are
+// rotated in interleaved pairs; the cache row is [keys of G heads | values of G heads].  A thread takes four dimensions of a
+// head at a time (heads are a multiple of 8 wide), which hold two whole pairs.
+constexpr int kRowsThreads = 256;
+template <typename T>
+__device__ __forceinline__ void ld4(const T* p, float* v);
+template <>
+__device__ __forceinline__ void ld4<float>(const float* p, float* v) {
+  const float4 t = *reinterpret_cast<const float4*>(p);
+  v[0] = t.x; v[1] = t.y; v[2] = t.z; v[3] = t.w;
+}
+template <>
+__device__ __forceinline__ void ld4<__nv_bfloat16>(const __nv_bfloat16* p, float* v) {
+  const uint2 t = *reinterpret_cast<const uint2*>(p);
+  v[0] = __uint_as_float(t.x << 16); v[1] = __uint_as_float(t.x & 0xffff0000u);
+  v[2] = __uint_as_float(t.y << 16); v[3] = __uint_as_float(t.y & 0xffff0000u);
+}
+template <typename T>
+__device__ __forceinline__ void st4(T* p, const float* v) {
+  Pair<T>::st(p, v[0], v[1]);
+  Pair<T>::st(p + 2, v[2], v[3]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kRowsThreads)
+proj_norm_rope_append_kernel(const T* __restrict__ in, long long in_rs, const float* __restrict__ qw, const float* __restrict__ kw,
+                             float q_count, float k_count, float eps, const float2* __restrict__ table, int table_len, int rot,
+                             T* __restrict__ q_out, long long q_rs, KvView kv, int row_w, const int* __restrict__ pos0,
+                             const int* __restrict__ slot0, const int* __restrict__ step_ptr, int Tn, int HD, int GD, int GE, int D,
+                             int* status) {
+  __shared__ float scratch[40], scratch2[40];
+  const long long tok = blockIdx.x;
+  const int s = (int)(tok / Tn), t = (int)(tok - (long long)s * Tn), tid = threadIdx.x;
+  const int step = step_ptr ? *step_ptr : 0;
+  const int pos = pos0[s] + step + t, slot = slot0[s] + step + t;
+  const int cap = kv.page_table ? kv.max_pages * kv.page_tokens : kv.page_tokens;
+  T* dst = nullptr;
+  if (slot >= 0 && slot < cap) {
+    const int lp = slot / kv.page_tokens;
+    long long pg = s;
+    if (kv.page_table) pg = kv.page_table[(long long)s * kv.max_pages + lp];
+    if (pg >= 0 && (kv.n_pages <= 0 || pg < kv.n_pages))
+      dst = static_cast<T*>(kv.k) + pg * kv.page_stride + (long long)(slot - lp * kv.page_tokens) * row_w;
+  }
+  const bool ok = pos >= 0 && pos < table_len;
+  if ((dst == nullptr || !ok) && tid == 0 && status) *status = 1;
+  const float2* cs = table + (long long)(ok ? pos : 0) * (rot >> 1);
+  const T* row = in + tok * in_rs;
+  const int n = HD + GD;
+  float qs = 0.f, ks = 0.f;
+  for (int c = tid * 4; c < n; c += kRowsThreads * 4) {
+    float v[4];
+    ld4<T>(row + c, v);
+    const float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
+    if (c < HD) qs += ss;
+    else ks += ss;
+  }
+  qs = block_sum(qs, scratch);
+  ks = block_sum(ks, scratch2);
+  const float qi = rsqrtf(qs / q_count + eps), ki = rsqrtf(ks / k_count + eps);
+  for (int c = tid * 4; c < n; c += kRowsThreads * 4) {
+    const bool is_q = c < HD;
+    const int x = is_q ? c : c - HD, d = x % D;
+    float v[4];
+    ld4<T>(row + c, v);  // in L1 from the first pass
+    const float4 w = *reinterpret_cast<const float4*>((is_q ? qw : kw) + x);
+    const float inv = is_q ? qi : ki;
+    v[0] *= inv * w.x; v[1] *= inv * w.y; v[2] *= inv * w.z; v[3] *= inv * w.w;
+#pragma unroll
+    for (int p = 0; p < 2; ++p) {
+      if (d + 2 * p < rot) {
+        const float2 f = cs[(d >> 1) + p];
+        const float a = v[2 * p], b = v[2 * p + 1];
+        v[2 * p] = a * f.x - b * f.y;
+        v[2 * p + 1] = b * f.x + a * f.y;
+      }
+    }
+    if (is_q) st4<T>(q_out + tok * q_rs + x, v);
+    else if (dst) st4<T>(dst + x, v);
+  }
+  if (dst) {
+    for (int c = tid * 4; c < GE; c += kRowsThreads * 4) {
+      float v[4];
+      ld4<T>(row + n + c, v);
+      st4<T>(dst + GD + c, v);
+    }
+  }
+}
+
 }  // namespace dgpt
 
 using namespace dgpt;
@@ -233,4 +323,38 @@ extern "C" int dgpt_rope_qknorm_kvappend(const void* q, const void* k, const voi
     return DGPT_E_UNSUPPORTED;
   }
   return launch_status("rope_qknorm_kvappend");
+}
+
+extern "C" int dgpt_proj_norm_rope_append(const void* in, int64_t in_row_stride, const float* q_weight, const float* k_weight,
+                                          int32_t q_count, int32_t k_count, float eps, const float* table, int32_t table_len,
+                                          int32_t rot_dims, void* q_out, int64_t q_out_row_stride, const dgpt_kv_layout* kv,
+                                          int32_t row_width, const int32_t* seq_pos0, const int32_t* seq_slot0,
+                                          const int32_t* step_ptr, int32_t n_seq, int32_t T, int32_t H, int32_t G, int32_t D,
+                                          int32_t Dv, int32_t dtype, int32_t* status, void* stream) {
+  DGPT_REQUIRE(in && q_weight && k_weight && table && q_out && seq_pos0 && seq_slot0, "proj_norm_rope_append: NULL pointer");
+  DGPT_REQUIRE(n_seq >= 0 && T >= 0 && H > 0 && G > 0 && D > 0 && D % 8 == 0 && Dv > 0 && Dv % 8 == 0 && q_count > 0 && k_count > 0,
+               "proj_norm_rope_append: bad sizes (heads must be a multiple of 8 wide)");
+  DGPT_REQUIRE(rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= D && table_len > 0, "proj_norm_rope_append: bad rotation");
+  DGPT_REQUIRE(in_row_stride % 8 == 0 && q_out_row_stride % 8 == 0 && row_width % 8 == 0 && row_width >= G * (D + Dv),
+               "proj_norm_rope_append: row strides must be multiples of 8");
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
+  DGPT_REQUIRE(al(in) && al(q_weight) && al(k_weight) && al(q_out), "proj_norm_rope_append: pointers must be 16-byte aligned");
+  if (int e = validate_kv(kv, D)) return e;
+  const long long n = (long long)n_seq * T;
+  if (n == 0) return DGPT_OK;
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const KvView view = make_view(kv);
+#define DGPT_PR(TT)                                                                                                         \
+  proj_norm_rope_append_kernel<TT><<<(unsigned)n, kRowsThreads, 0, st>>>(                                                   \
+      static_cast<const TT*>(in), in_row_stride, q_weight, k_weight, (float)q_count, (float)k_count, eps,                   \
+      reinterpret_cast<const float2*>(table), table_len, rot_dims, static_cast<TT*>(q_out), q_out_row_stride, view, row_width, \
+      seq_pos0, seq_slot0, step_ptr, T, H * D, G * D, G * Dv, D, status)
+  if (dtype == DGPT_F32) DGPT_PR(float);
+  else if (dtype == DGPT_BF16) DGPT_PR(__nv_bfloat16);
+  else {
+    set_error("proj_norm_rope_append: unknown dtype %d", dtype);
+    return DGPT_E_UNSUPPORTED;
+  }
+#undef DGPT_PR
+  return launch_status("proj_norm_rope_append");
 }

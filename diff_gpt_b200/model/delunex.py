@@ -24,18 +24,17 @@ query tokens expand keys and values with one GEMM and use the tensor-core attent
 
 from __future__ import annotations
 
-import contextlib
 import math
 from dataclasses import dataclass, field
 from typing import Callable
 
 import torch
-import torch.nn as nn
 import torch.nn.functional as F
 
 from .. import ops
 from .._lib import region
-from .gpt import DeviceModel, _sm_count
+from .configured import ConfiguredModel, fp32_reductions, round_up
+from .gpt import _sm_count
 from .kv_cache import LatentCache, PagedLatentCache
 
 EXPAND_MIN_TOKENS = 32  # query tokens per sequence from which keys and values are expanded
@@ -128,14 +127,10 @@ class DelunexConfig:
         return out
 
 
-def _up(n: int, m: int) -> int:
-    return -(-n // m) * m
-
-
 def padded_head(m: LatentAttention) -> int:
     """Head size the kernels work with: query, key and value heads are padded with zeros to one common size."""
     need = max(m.dim, m.vdim)
-    return next((d for d in EXPAND_HEAD_DIMS if d >= need), _up(need, 8))
+    return next((d for d in EXPAND_HEAD_DIMS if d >= need), round_up(need, 8))
 
 
 # ---- weights as the kernels want them ----------------------------------------------------
@@ -172,6 +167,10 @@ class _Packed:
     layers: list
     stamp: tuple
 
+    @property
+    def head(self) -> torch.Tensor:
+        return self.emb
+
 
 # ---- how one forward call is bound to cached state ------------------------------------------
 @dataclass
@@ -197,18 +196,6 @@ class LatentBinding:
     conv_in: torch.Tensor | None = None  # [n_layer, n_seq, taps - 1, C]
     conv_out: torch.Tensor | None = None
     fmha_impl: int = 0
-
-
-@contextlib.contextmanager
-def _fp32_reductions():
-    """bf16 products accumulate and reduce in fp32 (split-K partial sums included)."""
-    m = torch.backends.cuda.matmul
-    was = m.allow_bf16_reduced_precision_reduction
-    m.allow_bf16_reduced_precision_reduction = False
-    try:
-        yield
-    finally:
-        m.allow_bf16_reduced_precision_reduction = was
 
 
 def pick_latent_splits(rows: int, head_groups: int, keys: int) -> int:
@@ -316,7 +303,7 @@ class DelunexPlan:
     def run(self, ids32: torch.Tensor, b: LatentBinding, rows: torch.Tensor | None = None,
             tap: Callable[[int, torch.Tensor], None] | None = None) -> torch.Tensor | None:
         """`rows`: int32 places (among the n tokens) whose logits are wanted; `tap(i, x)` sees what leaves layer i."""
-        with _fp32_reductions():
+        with fp32_reductions():
             return self._run(ids32, b, rows, tap)
 
     def _run(self, ids32, b, rows, tap):
@@ -366,58 +353,27 @@ class DelunexPlan:
         return self.logits
 
 
-class Delunex(DeviceModel):
-    """Parameters are held under their checkpoint names with dots replaced (`l0.mix.q` -> `l0__mix__q`)."""
-
+class Delunex(ConfiguredModel):
     def __init__(self, config: DelunexConfig | dict, block_size: int = 32768) -> None:
         """`block_size` only bounds how far the Engine generates (the design has no positions)."""
         cfg = config if isinstance(config, DelunexConfig) else DelunexConfig.from_dict(config)
-        first = cfg.layers[0].mixer
-        super().__init__(block_size=block_size, vocab_size=cfg.vocab, n_embd=cfg.width, n_head=first.heads, n_layer=len(cfg.layers))
-        self.config = cfg
-        for name, shape in cfg.tensor_shapes().items():
-            self.register_parameter(name.replace(".", "__"), nn.Parameter(torch.zeros(shape), requires_grad=False))
-        self.ranks = {i: _up(l.mixer.kv_rank, 8) for i, l in enumerate(cfg.layers) if l.mixer.kv_from is None}
+        super().__init__(cfg, cfg.tensor_shapes(), block_size, cfg.vocab, cfg.width, cfg.layers[0].mixer.heads, len(cfg.layers))
+        self.ranks = {i: round_up(l.mixer.kv_rank, 8) for i, l in enumerate(cfg.layers) if l.mixer.kv_from is None}
         self.keep = max(l.mixer.window for l in cfg.layers) - 1
-        self._packed: _Packed | None = None
-        self._decode_plan: DelunexPlan | None = None  # the last single-token plan of `forward` / `logits_at`
-
-    @classmethod
-    def from_config(cls, config: dict) -> "Delunex":
-        return cls(config)
-
-    def load_tensors(self, tensors: dict) -> None:
-        want = self.config.tensor_shapes()
-        missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
-        if missing or extra:
-            raise ValueError(f"checkpoint does not fit the configuration: missing {missing[:4]}, unknown {extra[:4]}")
-        with torch.no_grad():
-            for name, shape in want.items():
-                if tuple(tensors[name].shape) != shape:
-                    raise ValueError(f"{name}: shape {tuple(tensors[name].shape)}, expected {shape}")
-                self.tensor(name).copy_(tensors[name])
-
-    def tensor(self, name: str) -> torch.Tensor:
-        return getattr(self, name.replace(".", "__"))
 
     # ---- weights -------------------------------------------------------------------------
-    def packed_weights(self) -> _Packed:
-        params = list(self.parameters())
-        stamp = tuple((p.data_ptr(), p._version, p.dtype) for p in params)
-        if self._packed is not None and self._packed.stamp == stamp:
-            return self._packed
+    def pack(self, stamp) -> _Packed:
         cfg = self.config
-        with torch.no_grad():
-            layers = [self._pack_layer(i) for i in range(len(cfg.layers))]
-            emb = self.embedding.detach()
-            final = self.tensor("final.norm").float() * cfg.logit_scale
-        self._packed = _Packed(emb=emb, one=torch.ones(1, device=emb.device), final_norm=final, layers=layers, stamp=stamp)
-        return self._packed
+        emb = self.embedding.detach()
+        return _Packed(
+            emb=emb, one=torch.ones(1, device=emb.device), final_norm=self.tensor("final.norm").float() * cfg.logit_scale,
+            layers=[self._pack_layer(i) for i in range(len(cfg.layers))], stamp=stamp,
+        )
 
     def _pack_layer(self, i: int) -> _PackedLayer:
         cfg = self.config
         m, ff = cfg.layers[i].mixer, cfg.layers[i].ff
-        C, H, D, r = cfg.width, m.heads, padded_head(m), _up(m.kv_rank, 8)
+        C, H, D, r = cfg.width, m.heads, padded_head(m), round_up(m.kv_rank, 8)
 
         def w(name):
             return self.tensor(f"l{i}.{name}").detach()
@@ -429,7 +385,7 @@ class Delunex(DeviceModel):
         parts = [heads(w("mix.q"), m.dim, C)]
         if own:
             parts.append(F.pad(w("mix.dkv"), (0, 0, 0, r - m.kv_rank)))
-        parts.append(F.pad(w("mix.g"), (0, 0, 0, _up(H, 8) - H)))
+        parts.append(F.pad(w("mix.g"), (0, 0, 0, round_up(H, 8) - H)))
         w_kv = torch.cat([heads(w("mix.uk"), m.dim, r), heads(w("mix.uv"), m.vdim, r)]).contiguous()
         w_o = F.pad(w("mix.o").view(C, H, m.vdim), (0, D - m.vdim)).reshape(C, H * D).contiguous()
         act = None
@@ -455,14 +411,6 @@ class Delunex(DeviceModel):
         )
 
     # ---- what the Engine needs -------------------------------------------------------------
-    @property
-    def embedding(self) -> torch.Tensor:
-        return self.embed
-
-    @property
-    def device_type(self) -> str:
-        return str(self.embed.device.type)
-
     def new_cache(self, batch_size: int = 1, seq_len: int = 0) -> LatentCache:
         emb = self.embedding
         cache = LatentCache(batch_size, self.ranks, self.keep, self.n_layer, self.config.taps, self.n_embd, emb.dtype, emb.device)
@@ -499,70 +447,19 @@ class Delunex(DeviceModel):
         )
         return bind, DelunexPlan(self, R, 1, want_logits=want_logits)
 
-    # ---- forward behind a cache ----------------------------------------------------------------
-    def _step(self, idx: torch.Tensor, cache: LatentCache, rows: torch.Tensor | None, tap=None) -> torch.Tensor:
-        B, T = idx.shape
-        dev = idx.device
-        assert cache.batch_size == B
-        cache.ensure(T)
+    def new_plan(self, n_seq, T, **kw) -> DelunexPlan:
+        return DelunexPlan(self, n_seq, T, **kw)
+
+    def step_binding(self, cache: LatentCache, B: int, T: int) -> LatentBinding:
+        dev = self.embedding.device
         slot = cache.slot
         start = torch.full((B,), slot, dtype=torch.int32, device=dev)
-        conv = cache.conv
-        bind = LatentBinding(
+        state = cache.state
+        return LatentBinding(
             layout=cache.layout, slot0=start, start1=torch.zeros_like(start), len1=start + 1, keys=slot + T, expand=True,
-            context=slot, latents=lambda layer, n: cache.span(layer, slot - n, slot + T), conv_in=conv.source,
-            conv_out=conv.source if T == 1 else conv.target,
+            context=slot, latents=lambda layer, n: cache.span(layer, slot - n, slot + T), conv_in=state.source["conv"],
+            conv_out=(state.source if T == 1 else state.target)["conv"],
         )
-        n_rows = B * T if rows is None else rows.numel()
-        plan = self._decode_plan
-        if T > 1 or plan is None or plan.n_seq != B or plan.xn.shape[0] != n_rows or plan.dt != self.embedding.dtype:
-            plan = DelunexPlan(self, B, T, rows=n_rows)
-            if T == 1:
-                self._decode_plan = plan
-        logits = plan.run(idx.reshape(-1).to(torch.int32), bind, None if rows is None else rows.to(torch.int32), tap)
-        if T > 1:
-            conv.flip()
-        cache.pos += T
-        if int(plan.status.item()):
-            raise RuntimeError(f"device-side status {int(plan.status.item())}: a cache slot was out of range, or a bounded wait ran out")
-        return logits
-
-    @torch.inference_mode()
-    def logits_at(self, idx, cache, rows):
-        return self._step(idx, cache, rows)
-
-    def forward(self, idx: torch.Tensor, targets: torch.Tensor | None = None, kv_cache: LatentCache | None = None):
-        if not idx.is_cuda:
-            raise RuntimeError("diff_gpt_b200.Delunex runs on CUDA only; there is no CPU path")
-        B, T = idx.shape
-        with torch.inference_mode():
-            cache = self.new_cache(B, T) if kv_cache is None else kv_cache
-            logits = self._step(idx, cache, None).view(B, T, self.vocab_size).clone()
-        loss = None
-        if targets is not None:
-            loss = F.cross_entropy(logits.view(-1, self.vocab_size).float(), targets.view(-1))
-        return logits, loss
-
-    @torch.inference_mode()
-    def generate(self, idx: torch.Tensor, max_new_tokens: int, sampler, seed: int | None = None):
-        """Prompt, then one token at a time through a cache."""
-        rng = None
-        if seed is not None:
-            rng = torch.Generator(device=idx.device)
-            rng.manual_seed(seed)
-        B, T = idx.shape
-        out = torch.zeros((B, T + max_new_tokens), dtype=torch.int64, device=idx.device)
-        out[:, :T] = idx
-        cache = self.new_cache(B, T + max_new_tokens)
-        new = idx
-        for cur in range(T, T + max_new_tokens):
-            logits = self(new, kv_cache=cache)[0][:, -1]
-            if sampler is not None:
-                new = sampler(logits, rng=rng).reshape(B, 1)
-            else:
-                new = torch.multinomial(F.softmax(logits.float(), dim=-1), num_samples=1, generator=rng)
-            out[:, cur] = new.reshape(-1)
-        return out
 
 
 def _softplus(v: float) -> float:

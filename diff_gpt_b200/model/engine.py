@@ -275,7 +275,7 @@ class DecodeRun:
         ops.step_advance(self.step, 1)
         if self.lmhead:
             ops.lmhead_sample(
-                self.plan.xn, self.packed.emb, self.tokens, cap=self.cap, temperature=self.temperature, top_p=self.top_p,
+                self.plan.xn, self.packed.head, self.tokens, cap=self.cap, temperature=self.temperature, top_p=self.top_p,
                 seed=self.seed, traj_ids=self.traj_ids, step=self.step, force_schedule=self.force,
                 force_group_rows=self.N, force_group_stride=self.G if self.force is not None else 0,
                 history_tokens=self.history, logits_out=self.head_logits, workspace=self.head_ws, status=self.plan.status,
@@ -306,7 +306,7 @@ class DecodeRun:
             self.plan.run(self.tokens, self.bind)
             if self.lmhead:  # and the head GEMM (function attributes, tensor-map encoder) into a scratch token buffer
                 ops.lmhead_sample(
-                    self.plan.xn, self.packed.emb, torch.empty_like(self.tokens), cap=self.cap, temperature=self.temperature,
+                    self.plan.xn, self.packed.head, torch.empty_like(self.tokens), cap=self.cap, temperature=self.temperature,
                     top_p=self.top_p, seed=self.seed, traj_ids=self.traj_ids, step=self.step, logits_out=self.head_logits,
                     workspace=self.head_ws, status=self.plan.status,
                 )

@@ -67,11 +67,12 @@ class DeviceModel(BaseGPT):
     @property
     @abstractmethod
     def embedding(self) -> torch.Tensor:
-        """The token table [V, C], which is also the output head; its device and dtype are the model's."""
+        """The token table [V, C]; its device and dtype are the model's."""
 
     @abstractmethod
     def packed_weights(self):
-        """Weights as the kernels want them; the same object until a parameter is modified or moved."""
+        """Weights as the kernels want them, `head` [V, C] (the output head; the token table where they are tied) among
+        them; the same object until a parameter is modified or moved."""
 
     # -- requests fed step by step --
     @abstractmethod
@@ -392,6 +393,10 @@ class _Packed:
     freqs_cis: torch.Tensor
     layers: list
     stamp: tuple
+
+    @property
+    def head(self) -> torch.Tensor:
+        return self.emb
 
 
 class GPT(DeviceModel):

@@ -14,6 +14,8 @@ and each trajectory owns a contiguous run of pages for the tokens it generates.
 
 from __future__ import annotations
 
+from dataclasses import dataclass
+
 import torch
 
 from .. import ops
@@ -171,57 +173,76 @@ class PagedKVCache:
         return self._layout(layer, self.row_table)
 
 
-class _ConvState:
-    """The last taps - 1 inputs of every layer's causal convolution, fp32 [n_layer, n_seq, taps - 1, width].
+@dataclass(frozen=True)
+class StateSpec:
+    """A tensor of per-sequence state: shape [lead, n_seq, *shape], `fill` before the first token."""
+
+    lead: int
+    shape: tuple[int, ...]
+    dtype: torch.dtype = torch.float32
+    fill: float = 0
+
+    def make(self, n_seq: int, device) -> torch.Tensor:
+        return torch.full((self.lead, n_seq, *self.shape), self.fill, dtype=self.dtype, device=device)
+
+
+class SeqState:
+    """What a model carries from token to token besides cached rows: convolution inputs, recurrent states, the last token.
 
     A forward over several tokens reads one buffer and writes the other (`source` / `target`, then `flip`), so that no
     thread overwrites what another still reads; one token at a time is updated in place.
     """
 
-    def __init__(self, n_layer: int, n_seq: int, taps: int, width: int, device) -> None:
-        self.buffers = torch.zeros((2, n_layer, n_seq, taps - 1, width), dtype=torch.float32, device=device)
+    def __init__(self, specs: dict[str, StateSpec], n_seq: int, device) -> None:
+        self.specs = specs
+        self.buffers = [{k: s.make(n_seq, device) for k, s in specs.items()} for _ in range(2)]
         self.current = 0
 
     @property
-    def source(self) -> torch.Tensor:
+    def source(self) -> dict[str, torch.Tensor]:
         return self.buffers[self.current]
 
     @property
-    def target(self) -> torch.Tensor:
+    def target(self) -> dict[str, torch.Tensor]:
         return self.buffers[1 - self.current]
 
     def flip(self) -> None:
         self.current = 1 - self.current
 
     def clear(self) -> None:
-        self.buffers.zero_()
+        for buf in self.buffers:
+            for k, t in buf.items():
+                t.fill_(self.specs[k].fill)
         self.current = 0
 
 
-class LatentCache:
-    """Cache of a sliding-window latent-attention model for requests fed step by step.
+class RowCache:
+    """Cache for requests fed step by step: one row of numbers per token and storage key (a latent, or the keys and values
+    of all heads), and the model's per-sequence state.
 
-    ranks      {layer: columns of a cached latent} for the layers that own a latent; other layers read an owner's
-    keep       tokens before a new one that some layer's window can still reach (the largest window less one), or None
-               when a layer sees everything
-    Latents live in one dense run of slots per sequence.  Only the last `keep` tokens are ever needed: when the run is
-    full they move to its front, and `base` (the position of slot 0) moves with them.  Keys carry no positions, so
-    slots are all that the attention kernels need.
+    widths      {key: columns of a row}, one entry per layer (or layer run) that caches rows
+    keep        tokens before a new one that some layer's window can still reach (the largest window less one), or None
+                when a layer sees everything
+    keep_first  first tokens that stay visible from every distance
+    Rows live in one dense run of slots per sequence.  Only the first `keep_first` and the last `keep` tokens are ever
+    needed: when the run is full the latter move to its front, behind the former, and `base` (how many tokens have been
+    dropped) moves with them.  Rows carry their positions in themselves where they have any, so slots are all that the
+    attention kernels need: a window counts slots back from the newest, and what was dropped lay behind every window.
     """
 
-    def __init__(self, batch_size: int, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int,
-                 dtype: torch.dtype, device) -> None:
-        self.batch_size, self.ranks, self.keep = batch_size, ranks, keep
+    def __init__(self, batch_size: int, widths: dict[int, int], keep: int | None, states: dict[str, StateSpec], dtype: torch.dtype,
+                 device, keep_first: int = 0) -> None:
+        self.batch_size, self.widths, self.keep, self.keep_first = batch_size, widths, keep, keep_first
         self.dtype, self.device = dtype, device
-        self.latents: dict[int, torch.Tensor] = {}
+        self.store: dict[int, torch.Tensor] = {}
         self.capacity = 0
-        self.conv = _ConvState(n_layer, batch_size, taps, width, device)
+        self.state = SeqState(states, batch_size, device)
         self.pos = 0
         self.base = 0
 
     def reset(self) -> None:
         self.pos = self.base = 0
-        self.conv.clear()
+        self.state.clear()
 
     def get_pos(self) -> int:
         return self.pos
@@ -235,87 +256,143 @@ class LatentCache:
         """Make room for T more tokens behind the ones that can still be seen."""
         if self.slot + T <= self.capacity:
             return
-        live = self.slot if self.keep is None else min(self.slot, self.keep)
+        fixed = min(self.slot, self.keep_first)
+        live = self.slot - fixed if self.keep is None else min(self.slot - fixed, self.keep)
         first = self.slot - live
-        if live + T <= self.capacity:
-            for t in self.latents.values():
-                t[:, :live] = t[:, first : first + live].clone()
+        if fixed + live + T <= self.capacity:
+            for t in self.store.values():
+                t[:, fixed : fixed + live] = t[:, first : first + live].clone()
         else:
             # room to slide in: as many slots again as stay live (at least 1024), so a move is paid for by many tokens
-            want = (live + T + max(live, 1024) + 63) // 64 * 64
-            for layer, r in self.ranks.items():
+            want = (fixed + live + T + max(live, 1024) + 63) // 64 * 64
+            for key, r in self.widths.items():
                 grown = torch.empty((self.batch_size, want, r), dtype=self.dtype, device=self.device)
-                if live:
-                    grown[:, :live] = self.latents[layer][:, first : first + live]
-                self.latents[layer] = grown
+                if fixed + live:
+                    grown[:, :fixed] = self.store[key][:, :fixed]
+                    grown[:, fixed : fixed + live] = self.store[key][:, first : first + live]
+                self.store[key] = grown
             self.capacity = want
-        self.base += first
+        self.base += first - fixed
 
-    def layout(self, layer: int) -> ops.KvLayout:
-        c = self.latents[layer]
+    def layout(self, key: int) -> ops.KvLayout:
+        c = self.store[key]
         return ops.kv_layout(c, c, page_stride=c.stride(0), head_stride=0, page_tokens=self.capacity)
 
-    def span(self, layer: int, first: int, end: int) -> torch.Tensor:
-        """Latents of slots [first, end) of all sequences as [batch * (end - first), r] (a copy if there are several)."""
-        c = self.latents[layer][:, first:end]
+    def kv_layout(self, key: int, D: int, v_col: int) -> ops.KvLayout:
+        """The same rows as separate keys and values of heads D wide, the values from column `v_col` on."""
+        c = self.store[key]
+        return ops.kv_layout(c, c[:, :, v_col:], page_stride=c.stride(0), head_stride=D, page_tokens=self.capacity)
+
+    def span(self, key: int, first: int, end: int) -> torch.Tensor:
+        """Rows of slots [first, end) of all sequences as [batch * (end - first), r] (a copy if there are several)."""
+        c = self.store[key][:, first:end]
         return c.reshape(-1, c.shape[-1])
 
 
-class PagedLatentCache:
-    """`PagedKVCache` for latent attention: per owning layer one pool of pages (n_pages, page_tokens, r).
+class PagedRowCache:
+    """`PagedKVCache` for cached rows: per storage key one pool of pages (n_pages, page_tokens, r).
 
     The prompt's pages are shared by a series' rows.  A row's own pages are a ring when every layer has a window: the
     table of a row maps each page of generated tokens to physical page (index mod ring length), and the ring is long
-    enough that the page being written is out of every window.  The convolutions' states are kept per series at the
-    prompt's end (`prompts`) and per row (`rows`).
+    enough that the page being written is out of every window.  Pages that may hold first tokens which stay visible (a
+    prompt can be shorter than `keep_first`) lie in front of the ring and are never written again.  The per-sequence state
+    is kept per series at the prompt's end (`prompts`) and per row (`states`).
     """
 
     prompts_exchangeable = False
 
-    def __init__(self, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int, n_series: int,
-                 rows_per_series: int, prefix_len: int, max_new: int, dtype: torch.dtype, device, page_tokens: int = 64) -> None:
+    def __init__(self, widths: dict[int, int], keep: int | None, states: dict[str, StateSpec], n_series: int, rows_per_series: int,
+                 prefix_len: int, max_new: int, dtype: torch.dtype, device, page_tokens: int = 64, keep_first: int = 0) -> None:
         pt = self.page_tokens = page_tokens
         self.n_series, self.rows_per_series = n_series, rows_per_series
         self.n_rows = n_series * rows_per_series
         self.prefix_len, self.max_new = prefix_len, max_new
         self.prefix_pages = max(1, -(-prefix_len // pt))
         self.own_pages = max(1, -(-max_new // pt))
-        self.ring_pages = self.own_pages if keep is None else min(self.own_pages, -(-keep // pt) + 1)
+        fixed = -(-max(0, keep_first - 1) // pt)  # a prompt has at least one token
+        self.ring_pages = self.own_pages if keep is None else min(self.own_pages, fixed + -(-keep // pt) + 1)
         n_pages = n_series * self.prefix_pages + self.n_rows * self.ring_pages
-        self.pools = {layer: torch.zeros((n_pages, pt, r), dtype=dtype, device=device) for layer, r in ranks.items()}
+        self.pools = {key: torch.zeros((n_pages, pt, r), dtype=dtype, device=device) for key, r in widths.items()}
         pre = torch.arange(n_series * self.prefix_pages, dtype=torch.int32).view(n_series, self.prefix_pages)
         ring = torch.arange(self.n_rows * self.ring_pages, dtype=torch.int32).view(self.n_rows, self.ring_pages)
-        own = n_series * self.prefix_pages + ring[:, torch.arange(self.own_pages) % self.ring_pages]
+        page = torch.arange(self.own_pages)
+        if self.ring_pages < self.own_pages:
+            page = torch.where(page < fixed, page, fixed + (page - fixed) % (self.ring_pages - fixed))
+        own = n_series * self.prefix_pages + ring[:, page]
         row = torch.cat([pre.repeat_interleave(rows_per_series, dim=0), own], dim=1)
         self.prefix_table = pre.contiguous().to(device)
         self.row_table = row.contiguous().to(device)
         self.suffix_slot0 = self.prefix_pages * pt
-        self.rows = torch.zeros((n_layer, self.n_rows, taps - 1, width), dtype=torch.float32, device=device)
-        self.prompts: list[tuple[torch.Tensor, torch.Tensor]] = []  # (series indices, their states at the prompt's end)
+        self.specs = states
+        self.states = {k: s.make(self.n_rows, device) for k, s in states.items()}
+        self.prompts: list[tuple[torch.Tensor, dict[str, torch.Tensor]]] = []  # (series indices, states at the prompt's end)
 
     @property
     def bytes(self) -> int:
         return sum(p.numel() * p.element_size() for p in self.pools.values())
 
-    def prompt_states(self, members: list[int]) -> torch.Tensor:
-        """The convolutions' states of the prompts of these series, [n_layer, len(members), taps - 1, width]."""
-        L, _, k, C = self.rows.shape
-        states = torch.zeros((L, len(members), k, C), dtype=torch.float32, device=self.rows.device)
-        self.prompts.append((torch.tensor(members, device=self.rows.device), states))
+    def prompt_states(self, members: list[int]) -> dict[str, torch.Tensor]:
+        """Where the prompts of these series leave their state, [lead, len(members), ...] each."""
+        dev = self.prefix_table.device
+        states = {k: s.make(len(members), dev) for k, s in self.specs.items()}
+        self.prompts.append((torch.tensor(members, device=dev), states))
         return states
 
     def begin_prompts(self) -> None:
         for _, states in self.prompts:
-            states.zero_()
+            for k, t in states.items():
+                t.fill_(self.specs[k].fill)
 
     def prompts_ready(self) -> None:
         """Every row starts from the state its series' prompt has left."""
-        L, _, k, C = self.rows.shape
-        rows = self.rows.view(L, self.n_series, self.rows_per_series, k, C)
         for members, states in self.prompts:
-            rows[:, members] = states.unsqueeze(2).expand(-1, -1, self.rows_per_series, -1, -1)
+            for k, t in states.items():
+                rows = self.states[k].view(t.shape[0], self.n_series, self.rows_per_series, *t.shape[2:])
+                rows[:, members] = t.unsqueeze(2).expand(-1, -1, self.rows_per_series, *t.shape[2:])
 
-    def layout(self, layer: int, table: torch.Tensor) -> ops.KvLayout:
-        p = self.pools[layer]
+    def layout(self, key: int, table: torch.Tensor) -> ops.KvLayout:
+        p = self.pools[key]
         return ops.kv_layout(p, p, page_stride=p.stride(0), head_stride=0, page_tokens=self.page_tokens, page_table=table,
                              n_pages=p.shape[0])
+
+    def kv_layout(self, key: int, table: torch.Tensor, D: int, v_col: int) -> ops.KvLayout:
+        """The same rows as separate keys and values of heads D wide, the values from column `v_col` on."""
+        p = self.pools[key]
+        return ops.kv_layout(p, p[:, :, v_col:], page_stride=p.stride(0), head_stride=D, page_tokens=self.page_tokens, page_table=table,
+                             n_pages=p.shape[0])
+
+
+# ---- the same for latents beside the inputs of causal convolutions ----------------------------------
+def conv_state(n_layer: int, taps: int, width: int) -> dict[str, StateSpec]:
+    """The last taps - 1 inputs of every layer's causal convolution, fp32 [n_layer, n_seq, taps - 1, width]."""
+    return {"conv": StateSpec(n_layer, (taps - 1, width))}
+
+
+class LatentCache(RowCache):
+    """ranks: {layer: columns of a cached latent} for the layers that own one; other layers read an owner's."""
+
+    def __init__(self, batch_size: int, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int,
+                 dtype: torch.dtype, device) -> None:
+        super().__init__(batch_size, ranks, keep, conv_state(n_layer, taps, width), dtype, device)
+
+    @property
+    def ranks(self) -> dict[int, int]:
+        return self.widths
+
+    @property
+    def latents(self) -> dict[int, torch.Tensor]:
+        return self.store
+
+
+class PagedLatentCache(PagedRowCache):
+    def __init__(self, ranks: dict[int, int], keep: int | None, n_layer: int, taps: int, width: int, n_series: int,
+                 rows_per_series: int, prefix_len: int, max_new: int, dtype: torch.dtype, device, page_tokens: int = 64) -> None:
+        super().__init__(ranks, keep, conv_state(n_layer, taps, width), n_series, rows_per_series, prefix_len, max_new, dtype, device,
+                         page_tokens)
+
+    @property
+    def rows(self) -> torch.Tensor:
+        return self.states["conv"]
+
+    def prompt_states(self, members: list[int]) -> torch.Tensor:
+        return super().prompt_states(members)["conv"]

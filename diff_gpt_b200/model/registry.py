@@ -14,8 +14,9 @@ import torch
 from ..weights import read_safetensors
 from .delunex import Delunex
 from .gpt import GPT, DeviceModel
+from .kipolix import Kipolix
 
-MODELS: dict[str, type[DeviceModel]] = {"GPT": GPT, "Delunex": Delunex}
+MODELS: dict[str, type[DeviceModel]] = {"GPT": GPT, "Delunex": Delunex, "Kipolix": Kipolix}
 
 
 def model_class(config: dict) -> type[DeviceModel]:

@@ -26,3 +26,14 @@ def apply_rotary_emb(x: torch.Tensor, freqs_cis: torch.Tensor) -> torch.Tensor:
     even, odd = pairs[..., 0], pairs[..., 1]
     rotated = torch.stack((even * cos - odd * sin, even * sin + odd * cos), dim=-1)
     return rotated.flatten(-2).to(x.dtype)
+
+
+def rotation_table(base: float, dims: int, positions: int, device) -> torch.Tensor:
+    """(cos, sin) of p * base^(-2 i / dims) as fp32 [positions, dims / 2, 2]; angles in float64, so that a table entry is
+    the nearest fp32 number whatever the position."""
+    p = torch.arange(positions, dtype=torch.float64, device=device)
+    f = torch.tensor(base, dtype=torch.float64, device=device) ** (
+        -2.0 * torch.arange(dims // 2, dtype=torch.float64, device=device) / max(dims, 1)
+    )
+    a = p[:, None] * f
+    return torch.stack([torch.cos(a), torch.sin(a)], dim=-1).to(torch.float32).contiguous()

@@ -268,21 +268,23 @@ def linear(
     swiglu: tuple[float, float] | None = None,
     add: torch.Tensor | None = None,
     xielu: tuple[float, float] | None = None,
+    silu_gate: bool = False,
     status: torch.Tensor | None = None,
 ) -> None:
     """out = a @ w.T on the tcgen05 kernel (bf16).  swiglu=(alpha, limit): the SwiGLU of interleaved column pairs is
     applied in the epilogue and `out` has half as many columns as `w` has rows.  add=r: out = r + a @ w.T, rounded
-    once (r may be `out`).  xielu=(alpha_p, alpha_n): that activation is applied in the epilogue."""
+    once (r may be `out`).  xielu=(alpha_p, alpha_n): that activation is applied in the epilogue.  silu_gate: column pairs
+    are (gate, up) and `out` = silu(gate) * up, half as many columns."""
     _cuda(a, w, out, add, status)
-    assert (swiglu is not None) + (add is not None) + (xielu is not None) <= 1
+    assert (swiglu is not None) + (add is not None) + (xielu is not None) + silu_gate <= 1
     M, K = a.shape
     N = w.shape[0]
     assert w.shape[1] == K and a.stride(1) == 1 and w.stride(1) == 1 and out.stride(1) == 1
-    assert out.shape == (M, N // 2 if swiglu else N) and a.dtype == w.dtype == out.dtype
+    assert out.shape == (M, N // 2 if swiglu or silu_gate else N) and a.dtype == w.dtype == out.dtype
     if add is not None:
         assert add.shape == out.shape and add.dtype == out.dtype and add.stride(1) == 1
     alpha, limit = swiglu or xielu or (0.0, 0.0)
-    epilogue = 1 if swiglu else 4 if xielu else 2 if add is not None else 0
+    epilogue = 1 if swiglu else 4 if xielu else 5 if silu_gate else 2 if add is not None else 0
     check(
         lib.dgpt_linear(
             a.data_ptr(), a.stride(0), w.data_ptr(), w.stride(0), out.data_ptr(), out.stride(0), _ptr(add),
@@ -733,3 +735,249 @@ def xielu(x: torch.Tensor, out: torch.Tensor, alpha_p: float, alpha_n: float) ->
     _cuda(x, out)
     assert x.is_contiguous() and out.is_contiguous() and x.shape == out.shape and x.dtype == out.dtype
     check(lib.dgpt_xielu(x.data_ptr(), out.data_ptr(), x.numel(), alpha_p, alpha_n, dtype_code(x), _stream()))
+
+
+def silu_mul(x: torch.Tensor, out: torch.Tensor) -> None:
+    """out = silu(x[:, 0::2]) * x[:, 1::2]"""
+    _cuda(x, out)
+    assert x.is_contiguous() and out.is_contiguous() and x.numel() == 2 * out.numel() and x.dtype == out.dtype
+    check(lib.dgpt_silu_mul(x.data_ptr(), out.data_ptr(), out.numel(), dtype_code(x), _stream()))
+
+
+# ---- grouped-query attention over cached rows, retention, several residual streams ---------------------
+def fmha_grouped(
+    q: torch.Tensor,
+    kv: KvLayout,
+    o: torch.Tensor,
+    *,
+    token_stride: int,
+    n_keys: int,
+    B: int,
+    H: int,
+    G: int,
+    D: int,
+    q_offset: int,
+    window: int,
+    keep_first: int,
+    scale: float,
+    impl: int = 0,
+    status: torch.Tensor | None = None,
+) -> None:
+    """q, o: [B * Tq, H * D] (2-D views with unit inner stride); kv: keys and values of G heads (see `dgpt_fmha_grouped`)."""
+    _cuda(q, o, status)
+    n = q.shape[0]
+    assert n % B == 0 and q.shape == o.shape == (n, H * D) and q.stride(1) == o.stride(1) == 1 and q.dtype == o.dtype
+    Tq = n // B
+    check(
+        lib.dgpt_fmha_grouped(
+            q.data_ptr(), Tq * q.stride(0), q.stride(0), C.byref(kv), token_stride, n_keys, o.data_ptr(), Tq * o.stride(0), o.stride(0),
+            B, H, G, Tq, D, q_offset, window, keep_first, scale, dtype_code(q), impl, _ptr(status), _stream(),
+        )
+    )
+
+
+def grouped_attn(
+    q: torch.Tensor,
+    kv: KvLayout,
+    len0: torch.Tensor | None,
+    start1: torch.Tensor,
+    len1: torch.Tensor,
+    step: torch.Tensor | None,
+    out: torch.Tensor,
+    *,
+    row_width: int,
+    v_col: int,
+    n_seq: int,
+    T: int,
+    H: int,
+    G: int,
+    dk: int,
+    dv: int,
+    window: int,
+    keep_first: int,
+    scale: float,
+    gate: torch.Tensor | None = None,
+    workspace: torch.Tensor | None = None,
+    n_splits: int = 1,
+    impl: int = 0,
+    status: torch.Tensor | None = None,
+) -> None:
+    """q: [n_seq * T, H * dk]; out: [n_seq * T, H * dv]; gate: [n_seq * T, H]."""
+    _cuda(q, len0, start1, len1, step, out, gate, workspace, status)
+    n = n_seq * T
+    assert q.shape == (n, H * dk) and out.shape == (n, H * dv) and q.stride(1) == out.stride(1) == 1 and q.dtype == out.dtype
+    assert gate is None or (gate.shape == (n, H) and gate.stride(1) == 1 and gate.dtype == q.dtype)
+    ws_bytes = 0 if workspace is None else workspace.numel() * workspace.element_size()
+    check(
+        lib.dgpt_grouped_attn(
+            q.data_ptr(), q.stride(0), C.byref(kv), row_width, v_col, _ptr(len0), start1.data_ptr(), len1.data_ptr(), _ptr(step),
+            _ptr(gate), 0 if gate is None else gate.stride(0), out.data_ptr(), out.stride(0), _ptr(workspace), ws_bytes, n_splits, n_seq,
+            T, H, G, dk, dv, window, keep_first, scale, dtype_code(q), impl, _ptr(status), _stream(),
+        )
+    )
+
+
+def proj_norm_rope_append(
+    x: torch.Tensor,
+    q_weight: torch.Tensor,
+    k_weight: torch.Tensor,
+    q_count: int,
+    k_count: int,
+    eps: float,
+    table: torch.Tensor,
+    q_out: torch.Tensor,
+    kv: KvLayout,
+    row_width: int,
+    pos0: torch.Tensor,
+    slot0: torch.Tensor,
+    step: torch.Tensor | None,
+    *,
+    n_seq: int,
+    T: int,
+    H: int,
+    G: int,
+    D: int,
+    Dv: int,
+    status: torch.Tensor | None = None,
+) -> None:
+    """x: [n_seq * T, >= H*D + G*(D + Dv)]; table: fp32 [positions, rot / 2, 2]; weights fp32 [H*D], [G*D]."""
+    _cuda(x, q_weight, k_weight, table, q_out, pos0, slot0, step, status)
+    assert x.shape[0] == q_out.shape[0] == n_seq * T and x.stride(1) == q_out.stride(1) == 1 and x.dtype == q_out.dtype
+    assert q_weight.dtype == k_weight.dtype == table.dtype == torch.float32 and table.is_contiguous() and table.dim() == 3
+    assert q_weight.numel() == H * D and k_weight.numel() == G * D and x.shape[1] >= H * D + G * (D + Dv)
+    assert pos0.dtype == slot0.dtype == torch.int32 and pos0.numel() == slot0.numel() == n_seq
+    check(
+        lib.dgpt_proj_norm_rope_append(
+            x.data_ptr(), x.stride(0), q_weight.data_ptr(), k_weight.data_ptr(), q_count, k_count, eps, table.data_ptr(),
+            table.shape[0], 2 * table.shape[1], q_out.data_ptr(), q_out.stride(0), C.byref(kv), row_width, pos0.data_ptr(),
+            slot0.data_ptr(), _ptr(step), n_seq, T, H, G, D, Dv, dtype_code(x), _ptr(status), _stream(),
+        )
+    )
+
+
+def retention_workspace_bytes(n_seq: int, T: int, H: int, dim: int, vdim: int) -> int:
+    return int(lib.dgpt_retention_workspace_bytes(n_seq, T, H, dim, vdim))
+
+
+def retention(
+    x: torch.Tensor,
+    cols: tuple[int, int, int, int],
+    table: torch.Tensor,
+    pos0: torch.Tensor,
+    step: torch.Tensor | None,
+    decay: torch.Tensor,
+    k_scale: float,
+    state_in: torch.Tensor | None,
+    state_out: torch.Tensor | None,
+    eps: float,
+    y: torch.Tensor,
+    workspace: torch.Tensor,
+    *,
+    n_seq: int,
+    T: int,
+    dim: int,
+    vdim: int,
+    impl: int = 0,
+    status: torch.Tensor | None = None,
+) -> None:
+    """x: [n_seq * T, *], q, k, v and gate from the four columns on; states: fp32 [n_seq, H, dim, vdim]; y: [n_seq * T, H * vdim]."""
+    _cuda(x, table, pos0, step, decay, state_in, state_out, y, workspace, status)
+    H = decay.numel()
+    assert x.shape[0] == y.shape[0] == n_seq * T and y.shape[1] == H * vdim and x.stride(1) == y.stride(1) == 1 and x.dtype == y.dtype
+    assert max(cols[0], cols[1]) + H * dim <= x.shape[1] and max(cols[2], cols[3]) + H * vdim <= x.shape[1]
+    assert table.dtype == decay.dtype == torch.float32 and table.is_contiguous() and table.dim() == 3 and decay.is_contiguous()
+    assert pos0.dtype == torch.int32 and pos0.numel() == n_seq
+    for t in (state_in, state_out):
+        assert t is None or (t.dtype == torch.float32 and t.is_contiguous() and t.numel() == n_seq * H * dim * vdim)
+    check(
+        lib.dgpt_retention(
+            x.data_ptr(), x.stride(0), *cols, table.data_ptr(), table.shape[0], 2 * table.shape[1], pos0.data_ptr(), _ptr(step),
+            decay.data_ptr(), k_scale, _ptr(state_in), _ptr(state_out), eps, y.data_ptr(), y.stride(0), workspace.data_ptr(),
+            workspace.numel() * workspace.element_size(), n_seq, T, H, dim, vdim, dtype_code(x), impl, _ptr(status), _stream(),
+        )
+    )
+
+
+def embed_streams(
+    ids: torch.Tensor,
+    prev_in: torch.Tensor | None,
+    prev_out: torch.Tensor | None,
+    emb: torch.Tensor,
+    big: torch.Tensor,
+    mul_prev: int,
+    mul_cur: int,
+    a: torch.Tensor,
+    w: torch.Tensor,
+    eps: float,
+    e: torch.Tensor,
+    h: torch.Tensor,
+    *,
+    n_seq: int,
+    T: int,
+) -> None:
+    """The bigram table has one row more than it has buckets; prev: int32 [n_seq], -1 = no token before."""
+    _cuda(ids, prev_in, prev_out, emb, big, a, w, e, h)
+    V, Cdim = emb.shape
+    assert ids.dtype == torch.int32 and ids.is_contiguous() and ids.numel() == n_seq * T and big.shape[1] == Cdim
+    assert emb.is_contiguous() and big.is_contiguous() and emb.dtype == big.dtype == h.dtype
+    assert e.shape == h.shape == (n_seq * T, Cdim) and e.dtype == a.dtype == w.dtype == torch.float32 and e.is_contiguous() and h.is_contiguous()
+    for t in (prev_in, prev_out):
+        assert t is None or (t.dtype == torch.int32 and t.numel() == n_seq and t.is_contiguous())
+    check(
+        lib.dgpt_embed_streams(
+            ids.data_ptr(), _ptr(prev_in), _ptr(prev_out), emb.data_ptr(), V, big.data_ptr(), big.shape[0] - 1, mul_prev, mul_cur,
+            a.data_ptr(), a.numel(), w.data_ptr(), eps, e.data_ptr(), h.data_ptr(), n_seq, T, Cdim, dtype_code(emb), _stream(),
+        )
+    )
+
+
+def _streams(x: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, y: torch.Tensor) -> int:
+    """Checks the streams [S, n, C] (or one row [n, C] that stands for all of them); returns their stride."""
+    S = out.numel()
+    assert x.dtype == mix.dtype == out.dtype == torch.float32 and mix.shape == (S, S) and mix.is_contiguous()
+    assert x.is_contiguous() and y.is_contiguous() and (x.shape == y.shape or x.shape == (S, *y.shape))
+    return 0 if x.dim() == 2 else x.stride(0)
+
+
+def streams_step(
+    x: torch.Tensor,
+    y: torch.Tensor,
+    mix: torch.Tensor,
+    out: torch.Tensor,
+    x_new: torch.Tensor,
+    a: torch.Tensor | None = None,
+    w: torch.Tensor | None = None,
+    eps: float = 0.0,
+    h: torch.Tensor | None = None,
+) -> None:
+    """x: fp32 [S, n, C], or [n, C] when all streams are equal; x_new: [S, n, C] (may be x); y, h: [n, C]."""
+    _cuda(x, y, mix, out, x_new, a, w, h)
+    stride = _streams(x, mix, out, y)
+    rows, Cdim = y.shape
+    S = out.numel()
+    assert x_new.shape == (S, rows, Cdim) and x_new.is_contiguous() and x_new.dtype == torch.float32
+    assert h is None or (h.shape == y.shape and h.dtype == y.dtype and h.is_contiguous() and a.numel() == S and w.numel() == Cdim)
+    check(
+        lib.dgpt_streams_step(
+            x.data_ptr(), stride, y.data_ptr(), mix.data_ptr(), out.data_ptr(), _ptr(a), S, _ptr(w), eps, x_new.data_ptr(),
+            x_new.stride(0), _ptr(h), rows, Cdim, dtype_code(y), _stream(),
+        )
+    )
+
+
+def streams_final(
+    x: torch.Tensor, y: torch.Tensor, mix: torch.Tensor, out: torch.Tensor, w: torch.Tensor, eps: float, h: torch.Tensor,
+    rows: torch.Tensor | None = None,
+) -> None:
+    """h = rms_norm(sum of the streams after the last sublayer) * w for the rows named by `rows` (None: the first ones)."""
+    _cuda(x, y, mix, out, w, h, rows)
+    stride = _streams(x, mix, out, y)
+    n, Cdim = y.shape
+    assert h.is_contiguous() and h.shape[1] == Cdim == w.numel() and h.dtype == y.dtype and w.dtype == torch.float32
+    assert rows is None or (rows.dtype == torch.int32 and rows.is_contiguous() and rows.numel() == h.shape[0])
+    check(
+        lib.dgpt_streams_final(
+            x.data_ptr(), stride, y.data_ptr(), mix.data_ptr(), out.data_ptr(), out.numel(), w.data_ptr(), eps, _ptr(rows),
+            h.data_ptr(), h.shape[0], n, Cdim, dtype_code(y), _stream(),
+        )
+    )

@@ -216,9 +216,10 @@ int dgpt_softcap(void* logits, int64_t n, float cap, int32_t dtype, void* stream
  *                the accumulator rounded to bf16 (as the reference's Linear output is)      out: [M, N / 2]
  *   epilogue 2:  out[m, n]     = resid[m, n] + acc[m, n], rounded once (resid may be out itself)   out: [M, N]
  *   epilogue 4:  out[m, n]     = xielu(acc[m, n]) with alpha_p = alpha, alpha_n = limit (see dgpt_xielu)   out: [M, N]
+ *   epilogue 5:  out[m, n / 2] = silu(acc[m, n]) * acc[m, n + 1] for even n, from the unrounded accumulator     out: [M, N / 2]
  * Replaces nn.Linear of src/diff_gpt/model/feed_forward.py:10-14 followed by swi_glu.py:11-19 (epilogue 1), any
  * bias-free nn.Linear of the path (epilogue 0), or a projection with the residual add that follows it
- * (src/diff_gpt/model/block.py:98-106, epilogue 2).  resid is ignored for epilogues 0, 1 and 4.  bf16 only; pointers 16-byte aligned, K and the row strides
+ * (src/diff_gpt/model/block.py:98-106, epilogue 2).  resid is ignored for epilogues 0, 1, 4 and 5.  bf16 only; pointers 16-byte aligned, K and the row strides
  * multiples of 8 elements, N a multiple of 16.  status: device int32, set non-zero if a bounded wait ran out. */
 int dgpt_linear(const void* a, int64_t a_row_stride, const void* w, int64_t w_row_stride, void* out,
                 int64_t out_row_stride, const void* resid, int64_t resid_row_stride, int32_t M, int32_t N,
@@ -354,6 +355,16 @@ int dgpt_fmha_window(const void* q, int64_t q_batch_stride, int64_t q_row_stride
                      int32_t H, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, float scale, int32_t dtype,
                      int32_t impl, int32_t* status, void* stream);
 
+/* Sliding-window attention over cached keys and values, grouped-query heads and first keys that stay visible: query i of a
+ * sequence sees key j when j <= q_offset + i and (q_offset + i - j < window, or window is 0, or j < keep_first); query head h
+ * reads key/value head h / (H / G).  kv: dense runs (page_table NULL, page_tokens = slots of a run, page_stride between
+ * sequences) or pages, with consecutive tokens of a head kv_token_stride elements apart; n_keys: keys of every sequence.
+ * Otherwise as dgpt_fmha_window. */
+int dgpt_fmha_grouped(const void* q, int64_t q_batch_stride, int64_t q_row_stride, const dgpt_kv_layout* kv,
+                      int64_t kv_token_stride, int32_t n_keys, void* o, int64_t o_batch_stride, int64_t o_row_stride, int32_t B,
+                      int32_t H, int32_t G, int32_t Tq, int32_t D, int32_t q_offset, int32_t window, int32_t keep_first,
+                      float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream);
+
 /* c = x / sqrt(mean(x[0..r_norm)^2) + eps) * w, rounded once and appended to a latent cache.  Token (s, t) goes to slot
  * seq_slot0[s] + step + t of sequence s; latent `slot` of a sequence lives at page * page_stride + (slot % page_tokens) * r
  * from kv->k_base (kv->v_base must name the same storage; head_stride is not used).  Columns r_norm..r-1 are written as
@@ -376,6 +387,21 @@ int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* 
                      const int32_t* len1, const int32_t* step_ptr, const void* gate, int64_t gate_row_stride, void* out,
                      int64_t out_row_stride, void* workspace, size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T,
                      int32_t H, int32_t r, int32_t window, float scale, int32_t dtype, int32_t impl, int32_t* status, void* stream);
+
+/* Grouped-query attention over cached rows [keys of G groups | values of G groups], with a sliding window and first tokens
+ * that stay visible:
+ *   out[row,h,:] = sigmoid(gate[row,h]) * sum_j p_j V(j,g),   p = softmax_j(q[row,h,:] . K(j,g) * scale),   g = h / (H / G)
+ * K(j,g) is columns [g*dk, +dk) of key j's row and V(j,g) columns [v_col + g*dv, +dv); rows are row_width elements apart
+ * from kv->k_base (kv->v_base must name the same storage; head_stride is not used).  Keys, ranges, splits, impl and status
+ * are those of dgpt_latent_attn, except that a row sees key i of 0 .. n-1 when i >= n - window (window 0: all) OR
+ * i < keep_first.  q: [n_seq*T, H*dk]; out: [n_seq*T, H*dv]; dk, dv, v_col and row_width multiples of 8.  Workspace from
+ * dgpt_latent_attn_workspace_bytes with r = dv. */
+int dgpt_grouped_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, int32_t row_width, int32_t v_col,
+                      const int32_t* len0, const int32_t* start1, const int32_t* len1, const int32_t* step_ptr,
+                      const void* gate, int64_t gate_row_stride, void* out, int64_t out_row_stride, void* workspace,
+                      size_t workspace_bytes, int32_t n_splits, int32_t n_seq, int32_t T, int32_t H, int32_t G, int32_t dk,
+                      int32_t dv, int32_t window, int32_t keep_first, float scale, int32_t dtype, int32_t impl,
+                      int32_t* status, void* stream);
 
 /* out = scale * emb[ids] in fp32.  ids: device int32 [n_tokens]; emb: [V, C] in dtype; out: fp32 [n_tokens, C]. */
 int dgpt_embed_scale(const int32_t* ids, const void* emb, float* out, int64_t n_tokens, int32_t C, int32_t V, float scale,
@@ -408,6 +434,60 @@ int dgpt_depth_avg_norm(const float* slab, int64_t term_stride, int32_t terms, c
 
 /* out[i] = alpha_p z^2 + z / 2 for z = in[i] > 0,  alpha_n (e^z - 1 - z) + z / 2 otherwise.  in, out: device [n] in dtype. */
 int dgpt_xielu(const void* in, void* out, int64_t n, float alpha_p, float alpha_n, int32_t dtype, void* stream);
+
+/* out[i] = silu(in[2 i]) * in[2 i + 1], silu(z) = z / (1 + e^-z).  in: [2 n_out]; out: [n_out], in dtype. */
+int dgpt_silu_mul(const void* in, void* out, int64_t n_out, int32_t dtype, void* stream);
+
+/* ---- several residual streams (hyper-connections), retention, norms over whole projections ------------------------ */
+
+/* e = emb[id] + big[row],  row = (previous id * mul_prev + id * mul_cur) mod buckets, or row `buckets` for a sequence's
+ * first token;  h = rms_norm((sum_s a[s]) e) * w: the combined input of the first sublayer when all S streams are e.
+ * ids: device int32 [n_seq * T]; prev_in: int32 [n_seq], the id before each sequence's first token of the call, -1 for none
+ * (NULL: none); prev_out: receives each sequence's last id, or NULL (may be prev_in only for T = 1); emb: [V, C] and big:
+ * [buckets + 1, C] in dtype; a: fp32 [S]; w: fp32 [C]; e_out: fp32 [n_seq * T, C]; h: dtype. */
+int dgpt_embed_streams(const int32_t* ids, const int32_t* prev_in, int32_t* prev_out, const void* emb, int32_t V, const void* big,
+                       int64_t buckets, int64_t mul_prev, int64_t mul_cur, const float* a, int32_t S, const float* w, float eps,
+                       float* e_out, void* h, int32_t n_seq, int32_t T, int32_t C, int32_t dtype, void* stream);
+
+/* One sublayer to the next:  x'_t = sum_s mix[s, t] x_s + out[t] y,   h = rms_norm(sum_t a[t] x'_t) * w.
+ * x, x_new: fp32 [rows, C] per stream, the streams `stride` elements apart (x_stream_stride 0: every stream is the same row;
+ * x_new may be x); y: [rows, C] in dtype; mix: fp32 [S, S]; out, a: fp32 [S]; w: fp32 [C]; h: dtype, or NULL.  S <= 16. */
+int dgpt_streams_step(const float* x, int64_t x_stream_stride, const void* y, const float* mix, const float* out, const float* a,
+                      int32_t S, const float* w, float eps, float* x_new, int64_t x_new_stream_stride, void* h, int64_t rows,
+                      int32_t C, int32_t dtype, void* stream);
+
+/* h[i] = rms_norm(sum_t x'_t) * w for the rows named by row_index (NULL: the first n_out of the n rows), x' as above. */
+int dgpt_streams_final(const float* x, int64_t x_stream_stride, const void* y, const float* mix, const float* out, int32_t S,
+                       const float* w, float eps, const int32_t* row_index, void* h, int64_t n_out, int64_t n, int32_t C,
+                       int32_t dtype, void* stream);
+
+/* Norm over whole projections, rotation, append.  Token (s, t), row n = s*T + t of `in`: columns [q: H*D | k: G*D | v: G*Dv].
+ *   q <- q / sqrt(sum(q^2) / q_count + eps) * q_weight over all H*D columns at once, k likewise (q_count, k_count: the
+ *   columns that count; the others are padding zeros),
+ *   then dimensions (2i, 2i+1), i < rot_dims / 2, of every head are rotated by table[position][i] = (cos, sin);
+ * q goes to q_out, [k | v] to cache row slot (row_width elements between rows, as in dgpt_grouped_attn).  position and slot
+ * are seq_pos0[s] and seq_slot0[s] + step + t.  table: device fp32 [table_len, rot_dims / 2, 2]; weights fp32, padded like
+ * the columns; status is set to 1 where a position or slot is out of range. */
+int dgpt_proj_norm_rope_append(const void* in, int64_t in_row_stride, const float* q_weight, const float* k_weight,
+                               int32_t q_count, int32_t k_count, float eps, const float* table, int32_t table_len,
+                               int32_t rot_dims, void* q_out, int64_t q_out_row_stride, const dgpt_kv_layout* kv,
+                               int32_t row_width, const int32_t* seq_pos0, const int32_t* seq_slot0, const int32_t* step_ptr,
+                               int32_t n_seq, int32_t T, int32_t H, int32_t G, int32_t D, int32_t Dv, int32_t dtype,
+                               int32_t* status, void* stream);
+
+/* Retention with a fixed decay per head:  S_t = decay[h] S_(t-1) + k_t v_t^T,  o_t = S_t^T q_t,
+ *   y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(g_t)                               per head, over its vdim columns
+ * q, k, v, g: columns q_col + h*dim, k_col + h*dim, v_col + h*vdim, g_col + h*vdim of row s*T + t of `in`.  q and k are rotated
+ * first: dimension i < rot_dims / 2 with i + rot_dims / 2 by table[pos0[s] + step + t][i] = (cos, sin); k is then multiplied
+ * by k_scale.  decay: device fp32 [H]; state_in / state_out: device fp32 [n_seq, H, dim, vdim] (NULL: zeros / not wanted; the
+ * same pointer only for T = 1); y: [n_seq*T, H*vdim] in dtype; workspace from the _bytes call, 16-byte aligned.
+ * impl: 0 = choose, 1 = recurrent, 2 = chunks on tcgen05 or fail.  status as elsewhere. */
+size_t dgpt_retention_workspace_bytes(int32_t n_seq, int32_t T, int32_t H, int32_t dim, int32_t vdim);
+int dgpt_retention(const void* in, int64_t in_row_stride, int32_t q_col, int32_t k_col, int32_t v_col, int32_t g_col,
+                   const float* table, int32_t table_len, int32_t rot_dims, const int32_t* pos0, const int32_t* step_ptr,
+                   const float* decay, float k_scale, const float* state_in, float* state_out, float eps, void* y,
+                   int64_t y_row_stride, float* workspace, size_t workspace_bytes, int32_t n_seq, int32_t T, int32_t H,
+                   int32_t dim, int32_t vdim, int32_t dtype, int32_t impl, int32_t* status, void* stream);
 
 #ifdef __cplusplus
 }
