@@ -1091,14 +1091,40 @@ def kernel_case(name: str, iters: int = 8) -> None:
 
 
 # ---------------------------------------------------------------------------------------
-# The Delunex design beside this package's GPT at equal size (--design delunex)
+# Model designs beside the closest other model of this package at equal size (--design): Delunex beside the GPT, Kipolix
+# beside Delunex
 # ---------------------------------------------------------------------------------------
-# layers of a real model's shape, a few of them; every other layer reads the latent of the one before
+# layers of a real model's shape, a few of them; in Delunex every other layer reads the latent of the one before
 DESIGN_SIZES = {
     "w1024": dict(width=1024, heads=16, dim=64, kv_rank=256, ff=4096, window=512, layers=8, vocab=16384),
     "w2048": dict(width=2048, heads=16, dim=128, kv_rank=512, ff=8192, window=1024, layers=8, vocab=16384),
     "w2048_long": dict(width=2048, heads=16, dim=128, kv_rank=256, ff=8192, window=4096, layers=8, vocab=16384),
 }
+
+
+# what Kipolix needs beside those: key/value heads, kept first tokens, retention heads (one layer in four is retention),
+# streams, and a gated feed-forward with the parameters of the plain one
+KIPOLIX_SIZES = {
+    "w1024": dict(kv_heads=4, keep=4, ret_heads=16, ret_dim=64, ret_vdim=64, streams=4, gated_ff=2736),
+    "w2048": dict(kv_heads=4, keep=4, ret_heads=16, ret_dim=128, ret_vdim=128, streams=4, gated_ff=5456),
+    "w2048_long": dict(kv_heads=8, keep=4, ret_heads=16, ret_dim=128, ret_vdim=128, streams=4, gated_ff=5456),
+}
+
+
+def kipolix_config(z: dict, k: dict) -> dict:
+    layers = []
+    for i in range(z["layers"]):
+        if i % 4 == 0:
+            n = k["ret_heads"]
+            m = dict(heads=n, dim=k["ret_dim"], vdim=k["ret_vdim"], rot={"dims": k["ret_dim"], "base": 1e4},
+                     decay=[1 - 2.0 ** (-5 - 6 * j / max(1, n - 1)) for j in range(n)])
+        else:
+            m = dict(heads=z["heads"], kv_heads=k["kv_heads"], dim=z["dim"], vdim=z["dim"], scale=z["dim"] ** -0.5,
+                     rot={"dims": z["dim"], "base": 1e4}, mask={"size": z["window"], "keep_first": k["keep"]})
+        layers.append({"type": "attention" if i % 4 else "retention", "mixer": m, "mlp": {"kind": "dense", "ff": k["gated_ff"]}})
+    return {"architecture": "Kipolix", "width": z["width"], "vocab": z["vocab"], "streams": k["streams"], "norm": {"eps": 1e-6},
+            "embedding": {"bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 31}}, "loop": {"start": 0, "stop": 0, "times": 1},
+            "layers": layers}
 
 
 def design_config(z: dict) -> dict:
@@ -1112,14 +1138,18 @@ def design_config(z: dict) -> dict:
             "embedding": {"scale": z["width"] ** 0.5}, "logit_scale": 1.0, "layers": layers}
 
 
-def design_model(kind: str, z: dict, dev):
-    """Random-weight model of the design or this package's GPT at the same width, heads, depth and vocabulary."""
-    from diff_gpt_b200 import Delunex, GPT
+def design_model(kind: str, name: str, dev):
+    """Random-weight model of a design or this package's GPT at the same width, heads, depth and vocabulary."""
+    from diff_gpt_b200 import Delunex, GPT, Kipolix
+
+    z = DESIGN_SIZES[name]
 
     g = torch.Generator(device=dev).manual_seed(1)
     with torch.device(dev):
         if kind == "delunex":
             m = Delunex(design_config(z))
+        elif kind == "kipolix":
+            m = Kipolix(kipolix_config(z, KIPOLIX_SIZES[name]))
         else:
             m = GPT(vocab_size=z["vocab"], n_embd=z["width"], n_head=z["heads"], n_layer=z["layers"], block_size=16384)
     m = m.to(torch.bfloat16).to(dev).eval()
@@ -1156,12 +1186,13 @@ def graph_ms(launch, iters: int) -> float:
     return event_ms(graph.replay, 3, 1) / iters
 
 
-def design_throughput(kind: str, z: dict, dev, rows: int, prompt: int, steps: int, prefill: tuple) -> dict:
+def design_throughput(kind: str, name: str, dev, rows: int, prompt: int, steps: int, prefill: tuple) -> dict:
     """Prefill (one plan, last-position logits) and decode (captured step, `rows` requests of `prompt` tokens each)."""
     from diff_gpt_b200 import TemperatureSampler, _lib
     from diff_gpt_b200.model.engine import DecodeRun
 
-    m = design_model(kind, z, dev)
+    z = DESIGN_SIZES[name]
+    m = design_model(kind, name, dev)
     g = torch.Generator(device=dev).manual_seed(2)
     out = {}
     with torch.inference_mode():
@@ -1192,29 +1223,25 @@ def design_throughput(kind: str, z: dict, dev, rows: int, prompt: int, steps: in
     return out
 
 
-def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
-    """Each hot kernel of the design alone, then the like kernel of the GPT, at one size: time, rate and fraction of the
-    measured peak.  Inputs larger than the L2, or several sets of them in turn."""
-    from diff_gpt_b200 import ops
+class KernelReport:
+    """Time, rate and fraction of the measured peak of one kernel at a time, by name in `out`."""
 
-    pk = peaks()
-    g = torch.Generator(device=dev).manual_seed(0)
-    bf, f32 = torch.bfloat16, torch.float32
-    C, H, D, r, W, ff = z["width"], z["heads"], z["dim"], z["kv_rank"], z["window"], z["ff"]
+    def __init__(self, dev) -> None:
+        self.dev, self.pk, self.out = dev, peaks(), {}
+        self.g = torch.Generator(device=dev).manual_seed(0)
 
-    def rnd(*s, dtype=bf):
-        return torch.randn(s, device=dev, generator=g, dtype=f32).to(dtype)
+    def rnd(self, *s, dtype=torch.bfloat16):
+        return torch.randn(s, device=self.dev, generator=self.g, dtype=torch.float32).to(dtype)
 
-    out = {}
-
-    def report(name, launch, iters, nbytes=None, flops=None):
-        ms = graph_ms(launch, iters)
+    def report(self, name, launch, iters, nbytes=None, flops=None):
+        pk, ms = self.pk, graph_ms(launch, iters)
         if flops is not None and (nbytes is None or flops / (pk["bf16_tflops"] * 1e12) > nbytes / (pk["hbm_gbs"] * 1e9)):
             rate, peak, unit = flops / ms / 1e9, pk["bf16_tflops"], "TFLOP/s"
         else:
             rate, peak, unit = nbytes / ms / 1e6, pk["hbm_gbs"], "GB/s"
-        out[name] = {"us": 1e3 * ms, "rate": rate, "unit": unit, "frac": rate / peak}
+        self.out[name] = {"us": 1e3 * ms, "rate": rate, "unit": unit, "frac": rate / peak}
 
+    @staticmethod
     def in_turn(sets, fn):
         turn = [0]
 
@@ -1224,8 +1251,102 @@ def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
 
         return launch
 
+    @staticmethod
     def copies(nbytes):  # sets of inputs that together are well beyond the 126 MB L2
         return max(1, min(16, -(-400_000_000 // nbytes)))
+
+
+def kipolix_kernels(z: dict, k: dict, dev, rows: int, T: int) -> dict:
+    """Each hot kernel of Kipolix alone at one size (see `design_kernels` for the like kernels of the other designs)."""
+    from diff_gpt_b200 import ops
+    from diff_gpt_b200.model.delunex import pick_latent_splits
+    from diff_gpt_b200.model.rope import rotation_table
+
+    R = KernelReport(dev)
+    rnd, report, in_turn, copies = R.rnd, R.report, R.in_turn, R.copies
+    bf, f32 = torch.bfloat16, torch.float32
+    C, H, D, W, ff, G, keep, S = z["width"], z["heads"], z["dim"], z["window"], k["gated_ff"], k["kv_heads"], k["keep"], k["streams"]
+    st = torch.zeros(1, dtype=torch.int32, device=dev)
+    i32 = lambda n, v: torch.full((n,), v, dtype=torch.int32, device=dev)  # noqa: E731
+    tab = rotation_table(1e4, D, max(T, 4 * W), dev)
+    # ---- decode attention: rows x (W + kept) keys out of a longer context ----
+    width, n_ctx, pt = 2 * G * D, W + 1024, 64
+    per = -(-n_ctx // pt)
+    pool = rnd(rows * per, pt, width)
+    table = torch.randperm(rows * per, device=dev, generator=R.g).to(torch.int32).view(rows, per)
+    lay = ops.kv_layout(pool, pool, pt * width, 0, pt, table, n_pages=rows * per)
+    q, o = rnd(rows, H * D), torch.empty((rows, H * D), device=dev, dtype=bf)
+    splits = pick_latent_splits(rows, G, W + keep)
+    ws = torch.empty(max(4, ops.latent_attn_workspace_bytes(rows, H, D, splits) // 4), device=dev) if splits > 1 else None
+    i0, n1 = i32(rows, 0), i32(rows, n_ctx)
+    report("grouped_attn", lambda: ops.grouped_attn(q, lay, None, i0, n1, None, o, row_width=width, v_col=G * D, n_seq=rows, T=1, H=H, G=G, dk=D,
+                                                    dv=D, window=W, keep_first=keep, scale=D**-0.5, workspace=ws, n_splits=splits, status=st),
+           8, rows * ((W + keep) * width + 2 * H * D) * 2, 4 * rows * H * W * D)
+    del pool
+    # ---- prefill attention ----
+    kv = rnd(1, T, width)
+    lay = ops.kv_layout(kv, kv[:, :, G * D :], kv.stride(0), D, T)
+    q, o = rnd(T, H * D), torch.empty((T, H * D), device=dev, dtype=bf)
+    seen = T * W - W * (W - 1) // 2 + max(0, T - W) * keep if T >= W else T * (T + 1) // 2
+    report("fmha_grouped", lambda: ops.fmha_grouped(q, lay, o, token_stride=width, n_keys=T, B=1, H=H, G=G, D=D, q_offset=0, window=W, keep_first=keep,
+                                                    scale=D**-0.5, status=st), 8, None, 4 * D * H * seen)
+    # ---- retention ----
+    n, d, e = k["ret_heads"], k["ret_dim"], k["ret_vdim"]
+    cols = (0, n * d, 2 * n * d, 2 * n * d + n * e)
+    decay = torch.tensor([1 - 2.0 ** (-5 - 6 * j / max(1, n - 1)) for j in range(n)], device=dev)
+    rtab = rotation_table(1e4, d, T, dev)
+    for B, t in ((1, T), (8, T // 4)):
+        x, y = rnd(B * t, 2 * n * (d + e)), torch.empty((B * t, n * e), device=dev, dtype=bf)
+        so = torch.empty(B, n, d, e, device=dev)
+        rws = torch.empty(ops.retention_workspace_bytes(B, t, n, d, e) // 4, device=dev)
+        z0 = i32(B, 0)
+        report(f"retention_{B}x{t}", lambda: ops.retention(x, cols, rtab, z0, None, decay, 0.96, d**-0.5, None, so, 1e-6, y, rws, n_seq=B, T=t, dim=d,
+                                                           vdim=e, status=st),
+               8, B * t * n * (2 * d + 3 * e) * 2, 2 * B * t * n * (128 * (d + e) + 2 * d * e))
+    sets = [(rnd(rows, 2 * n * (d + e)), rnd(rows, n, d, e, dtype=f32), torch.empty((rows, n * e), device=dev, dtype=bf))
+            for _ in range(copies(8 * rows * n * d * e))]
+    rws, z0 = torch.empty(ops.retention_workspace_bytes(rows, 1, n, d, e) // 4, device=dev), i32(rows, 77)
+    report("retention_decode", in_turn(sets, lambda xx, ss, yy: ops.retention(xx, cols, rtab, z0, None, decay, 0.96, d**-0.5, ss, ss, 1e-6, yy, rws,
+                                                                             n_seq=rows, T=1, dim=d, vdim=e, status=st)),
+           8, rows * n * (8 * d * e + 2 * (2 * d + 3 * e)))
+    del sets
+    # ---- streams, embedding, append ----
+    mix, out, a, w = torch.eye(S, device=dev), rnd(S, dtype=f32), rnd(S, dtype=f32), rnd(C, dtype=f32)
+    xs, y, h = rnd(S, T, C, dtype=f32), rnd(T, C), rnd(T, C)
+    xn = torch.empty_like(xs)
+    report("streams_step", lambda: ops.streams_step(xs, y, mix, out, xn, a, w, 1e-6, h), 8, T * C * (8 * S + 4))
+    del xn
+    small = [(rnd(S, rows, C, dtype=f32), rnd(rows, C), rnd(rows, C)) for _ in range(copies(rows * C * (4 * S + 4)))]
+    report("streams_step_decode", in_turn(small, lambda xx, yy, hh: ops.streams_step(xx, yy, mix, out, xx, a, w, 1e-6, hh)), 16,
+           rows * C * (8 * S + 4))
+    del small, xs
+    emb, big, ids = rnd(z["vocab"], C), rnd(65522, C), torch.randint(0, z["vocab"], (T,), device=dev, generator=R.g, dtype=torch.int32)
+    ef = torch.empty((T, C), device=dev)
+    report("embed_streams", lambda: ops.embed_streams(ids, None, None, emb, big, 8191, 31, a, w, 1e-6, ef, h, n_seq=1, T=T), 8, T * C * 10)
+    del emb, big
+    proj = rnd(T, H * D + width)
+    qw, kw = rnd(H * D, dtype=f32), rnd(G * D, dtype=f32)
+    ll = ops.kv_layout(kv, kv, kv.stride(0), 0, T)
+    z1 = i32(1, 0)
+    report("proj_norm_rope_append", lambda: ops.proj_norm_rope_append(proj, qw, kw, H * D, G * D, 1e-6, tab, q, ll, width, z1, z1, None, n_seq=1, T=T,
+                                                                      H=H, G=G, D=D, Dv=D, status=st), 8, T * (H * D + width) * 4)
+    # ---- feed-forward GEMM with the gate ----
+    wgu, act, full = rnd(2 * ff, C), torch.empty((T, ff), device=dev, dtype=bf), torch.empty((T, 2 * ff), device=dev, dtype=bf)
+    report("linear_silu_gate", lambda: ops.linear(h, wgu, act, silu_gate=True, status=st), 8, None, 4 * T * ff * C)
+    report("cublas_gate_up", lambda: torch.mm(h, wgu.t(), out=full), 8, None, 4 * T * ff * C)
+    assert int(st.item()) == 0
+    return R.out
+
+
+def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
+    """Each hot kernel of the design alone, then the like kernel of the GPT, at one size: time, rate and fraction of the
+    measured peak.  Inputs larger than the L2, or several sets of them in turn."""
+    from diff_gpt_b200 import ops
+
+    R = KernelReport(dev)
+    g, rnd, report, in_turn, copies = R.g, R.rnd, R.report, R.in_turn, R.copies
+    bf, f32 = torch.bfloat16, torch.float32
+    C, H, D, r, W, ff = z["width"], z["heads"], z["dim"], z["kv_rank"], z["window"], z["ff"]
 
     st = torch.zeros(1, dtype=torch.int32, device=dev)
     # ---- decode attention over latents: rows x W keys ----
@@ -1310,7 +1431,7 @@ def design_kernels(z: dict, dev, rows: int, T: int) -> dict:
     gate = rnd(T, C)
     report("gpt.sigmoid_gate", lambda: ops.sigmoid_gate(qo, gate), 8, T * C * 2 * 3)
     assert int(st.item()) == 0
-    return out
+    return R.out
 
 
 def run_design(args) -> None:
@@ -1322,12 +1443,17 @@ def run_design(args) -> None:
     for name in names:
         z = DESIGN_SIZES[name]
         rows, prompt, T = 256, 2 * z["window"] if z["window"] <= 1024 else z["window"], 8192
-        entry = {"config": z}
+        entry = {"config": {**z, **(KIPOLIX_SIZES[name] if args.design == "kipolix" else {})}}
         if not args.kernels_only:
-            for kind in ("delunex", "gpt"):
-                entry[kind] = design_throughput(kind, z, dev, rows, prompt, 32, ((1, T), (8, 2048)))
+            for kind in ("kipolix", "delunex") if args.design == "kipolix" else ("delunex", "gpt"):
+                entry[kind] = design_throughput(kind, name, dev, rows, prompt, 32, ((1, T), (8, 2048)))
                 torch.cuda.empty_cache()
-        entry["kernels"] = design_kernels(z, dev, rows, T)
+        entry["kernels"] = {}
+        if args.design == "kipolix":
+            entry["kernels"] = kipolix_kernels(z, KIPOLIX_SIZES[name], dev, rows, T)
+            torch.cuda.empty_cache()
+        if not args.own_kernels:
+            entry["kernels"].update(design_kernels(z, dev, rows, T))
         torch.cuda.empty_cache()
         line["sizes"][name] = entry
     line["clocks"] = clocks.stop()
@@ -1354,11 +1480,12 @@ def main() -> None:
     ap.add_argument("--no-graph", action="store_true", help="launch the decode steps eagerly (for profilers)")
     ap.add_argument("--small", action="store_true",
                     help="profiling case: 2048 trajectories x 64 steps (4.8 GB of KV), same model and prompt")
-    ap.add_argument("--design", default=None, choices=["delunex"],
-                    help="instead of the workload above: prefill and decode throughput of this model design beside the GPT at "
-                         "equal size, and its kernels beside the GPT's like ones; one JSON line")
+    ap.add_argument("--design", default=None, choices=["delunex", "kipolix"],
+                    help="instead of the workload above: prefill and decode throughput of this model design beside the closest other "
+                         "model at equal size (delunex: the GPT; kipolix: Delunex), and its kernels beside the like ones; one JSON line")
     ap.add_argument("--sizes", default=None, help="with --design: comma-separated names out of " + ", ".join(DESIGN_SIZES))
     ap.add_argument("--kernels-only", action="store_true", help="with --design: the kernel table alone")
+    ap.add_argument("--own-kernels", action="store_true", help="with --design kipolix: leave the like kernels of the other designs out")
     args = ap.parse_args()
     if args.small:
         globals().update(TRAJECTORIES=2048, HORIZON=64)

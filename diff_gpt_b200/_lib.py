@@ -122,7 +122,7 @@ PROTOTYPES = {
     "dgpt_retention_workspace_bytes": (_sz, [_i32, _i32, _i32, _i32, _i32]),
     "dgpt_retention": (
         C.c_int,
-        [_p, _i64, _i32, _i32, _i32, _i32, _p, _i32, _i32, _p, _p, _p, _f32, _p, _p, _f32, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32,
+        [_p, _i64, _i32, _i32, _i32, _i32, _p, _i32, _i32, _p, _p, _p, _f32, _f32, _p, _p, _f32, _p, _i64, _p, _sz, _i32, _i32, _i32, _i32,
          _i32, _i32, _i32, _p, _p],
     ),
     "dgpt_embed_scale": (C.c_int, [_p, _p, _p, _i64, _i32, _i32, _f32, _i32, _p]),

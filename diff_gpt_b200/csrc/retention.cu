@@ -194,6 +194,14 @@ static int ret_max_smem() {
 }
 
 template <typename T>
+static int head_norm_gate(const RetentionArgs& a, cudaStream_t st) {
+  const long long n = (long long)a.n_seq * a.Tn;
+  head_norm_gate_kernel<T><<<(unsigned)((n * a.H + 7) / 8), 256, 0, st>>>(a.o, static_cast<const T*>(a.in) + a.g_col, a.in_rs, a.eps,
+                                                                          static_cast<T*>(a.y), a.y_rs, n, a.H, a.vdim);
+  return launch_status("head_norm_gate");
+}
+
+template <typename T>
 static int retention_recurrent(const RetentionArgs& a, cudaStream_t st) {
   const int e = a.vdim;
   auto vec_ok = [&](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
@@ -223,11 +231,10 @@ static int retention_recurrent(const RetentionArgs& a, cudaStream_t st) {
   const dim3 grid((unsigned)(a.n_seq * a.H), (unsigned)((e + es - 1) / es));
   retention_scan_kernel<T><<<grid, kRetThreads, need(es), st>>>(a, es);
   if (int x = launch_status("retention_scan")) return x;
-  const long long n = (long long)a.n_seq * a.Tn;
-  head_norm_gate_kernel<T><<<(unsigned)((n * a.H + 7) / 8), 256, 0, st>>>(a.o, static_cast<const T*>(a.in) + a.g_col, a.in_rs, a.eps,
-                                                                          static_cast<T*>(a.y), a.y_rs, n, a.H, e);
-  return launch_status("head_norm_gate");
+  return head_norm_gate<T>(a, st);
 }
+
+constexpr int kRetChunkMin = 16;  // tokens per sequence from which the chunked form is faster than walking through them
 
 }  // namespace dgpt
 
@@ -235,8 +242,8 @@ using namespace dgpt;
 
 extern "C" int dgpt_retention(const void* in, int64_t in_row_stride, int32_t q_col, int32_t k_col, int32_t v_col, int32_t g_col,
                               const float* table, int32_t table_len, int32_t rot_dims, const int32_t* pos0, const int32_t* step_ptr,
-                              const float* decay, float k_scale, const float* state_in, float* state_out, float eps, void* y,
-                              int64_t y_row_stride, float* workspace, size_t workspace_bytes, int32_t n_seq, int32_t T, int32_t H,
+                              const float* decay, float min_decay, float k_scale, const float* state_in, float* state_out,
+                              float eps, void* y, int64_t y_row_stride, float* workspace, size_t workspace_bytes, int32_t n_seq, int32_t T, int32_t H,
                               int32_t dim, int32_t vdim, int32_t dtype, int32_t impl, int32_t* status, void* stream) {
   DGPT_REQUIRE(in && table && pos0 && decay && y, "retention: NULL pointer");
   DGPT_REQUIRE(n_seq >= 0 && T >= 0 && H > 0 && dim > 0 && vdim > 0 && rot_dims >= 0 && rot_dims % 2 == 0 && rot_dims <= dim && table_len > 0,
@@ -266,10 +273,22 @@ extern "C" int dgpt_retention(const void* in, int64_t in_row_stride, int32_t q_c
     set_error("retention: a 16-byte aligned workspace of %zu bytes is needed, %zu given", need, workspace_bytes);
     return DGPT_E_WORKSPACE;
   }
+  const bool tc_ok = retention_tc_supported(a, dtype, min_decay);
+  if (impl == 2 && !tc_ok) {
+    set_error("retention: the chunked form covers bf16 with key sizes up to 128, sizes and columns that are multiples of 8 and decays "
+              "from 1/16 on (dtype %d, sizes %d and %d, smallest decay %g)", dtype, dim, vdim, (double)min_decay);
+    return DGPT_E_UNSUPPORTED;
+  }
+  if (tc_ok && (impl == 2 || (impl == 0 && T >= kRetChunkMin))) {
+    const size_t o_bytes = ((size_t)n_seq * T * H * vdim * sizeof(float) + 15) & ~(size_t)15;
+    if (int e = retention_tc_launch(a, workspace + o_bytes / sizeof(float), st)) return e;
+    return vdim > 128 ? head_norm_gate<__nv_bfloat16>(a, st) : DGPT_OK;
+  }
   return dtype == DGPT_F32 ? retention_recurrent<float>(a, st) : retention_recurrent<__nv_bfloat16>(a, st);
 }
 
 extern "C" size_t dgpt_retention_workspace_bytes(int32_t n_seq, int32_t T, int32_t H, int32_t dim, int32_t vdim) {
-  (void)dim;
-  return (((size_t)n_seq * T * H * vdim * sizeof(float)) + 15) & ~(size_t)15;
+  if (n_seq <= 0 || T <= 0 || H <= 0 || dim <= 0 || vdim <= 0) return 16;
+  // o where it waits for its norm, then the states of the chunked form's segments
+  return ((((size_t)n_seq * T * H * vdim * sizeof(float)) + 15) & ~(size_t)15) + retention_tc_workspace_bytes(n_seq, T, H, dim, vdim);
 }

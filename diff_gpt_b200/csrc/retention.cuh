@@ -25,4 +25,10 @@ struct RetentionArgs {
   int* status;
 };
 
+// chunked form (retention_tc.cu): bf16, dim <= 128, decays (the smallest: min_decay) that leave a chunk room.  With several
+// slices of value columns it leaves o in a.o, unnormalised; otherwise y is written.
+bool retention_tc_supported(const RetentionArgs& a, int dtype, float min_decay);
+size_t retention_tc_workspace_bytes(int n_seq, int T, int H, int dim, int vdim);
+int retention_tc_launch(const RetentionArgs& a, float* seg_state, cudaStream_t st);
+
 }  // namespace dgpt

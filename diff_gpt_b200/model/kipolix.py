@@ -294,7 +294,7 @@ class KipolixPlan:
         ws = self._buf("ret_ws", max(4, ops.retention_workspace_bytes(n_seq, T, m.heads, m.dim, m.vdim) // 4), dtype=torch.float32)
         name = f"ret{run}"
         ops.retention(
-            proj, lw.cols, b.tables[m.rot.base, m.rot.dims], b.pos0, b.step, lw.decay, m.dim**-0.5,
+            proj, lw.cols, b.tables[m.rot.base, m.rot.dims], b.pos0, b.step, lw.decay, min(m.decay), m.dim**-0.5,
             None if b.state_in is None else b.state_in[name], b.state_out[name], self.model.config.eps, y, ws, n_seq=n_seq, T=T,
             dim=m.dim, vdim=m.vdim, status=self.status,
         )

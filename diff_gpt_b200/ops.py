@@ -866,6 +866,7 @@ def retention(
     pos0: torch.Tensor,
     step: torch.Tensor | None,
     decay: torch.Tensor,
+    min_decay: float,
     k_scale: float,
     state_in: torch.Tensor | None,
     state_out: torch.Tensor | None,
@@ -892,7 +893,7 @@ def retention(
     check(
         lib.dgpt_retention(
             x.data_ptr(), x.stride(0), *cols, table.data_ptr(), table.shape[0], 2 * table.shape[1], pos0.data_ptr(), _ptr(step),
-            decay.data_ptr(), k_scale, _ptr(state_in), _ptr(state_out), eps, y.data_ptr(), y.stride(0), workspace.data_ptr(),
+            decay.data_ptr(), min_decay, k_scale, _ptr(state_in), _ptr(state_out), eps, y.data_ptr(), y.stride(0), workspace.data_ptr(),
             workspace.numel() * workspace.element_size(), n_seq, T, H, dim, vdim, dtype_code(x), impl, _ptr(status), _stream(),
         )
     )

@@ -394,7 +394,8 @@ int dgpt_latent_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* 
  * K(j,g) is columns [g*dk, +dk) of key j's row and V(j,g) columns [v_col + g*dv, +dv); rows are row_width elements apart
  * from kv->k_base (kv->v_base must name the same storage; head_stride is not used).  Keys, ranges, splits, impl and status
  * are those of dgpt_latent_attn, except that a row sees key i of 0 .. n-1 when i >= n - window (window 0: all) OR
- * i < keep_first.  q: [n_seq*T, H*dk]; out: [n_seq*T, H*dv]; dk, dv, v_col and row_width multiples of 8.  Workspace from
+ * i < keep_first.  q: [n_seq*T, H*dk]; out: [n_seq*T, H*dv]; dk, dv, v_col and row_width multiples of 8; every
+ * column of a row that has been written holds a finite number (also those outside keys and values).  Workspace from
  * dgpt_latent_attn_workspace_bytes with r = dv. */
 int dgpt_grouped_attn(const void* q, int64_t q_row_stride, const dgpt_kv_layout* kv, int32_t row_width, int32_t v_col,
                       const int32_t* len0, const int32_t* start1, const int32_t* len1, const int32_t* step_ptr,
@@ -479,14 +480,14 @@ int dgpt_proj_norm_rope_append(const void* in, int64_t in_row_stride, const floa
  *   y_t = o_t / sqrt(mean(o_t^2) + eps) * silu(g_t)                               per head, over its vdim columns
  * q, k, v, g: columns q_col + h*dim, k_col + h*dim, v_col + h*vdim, g_col + h*vdim of row s*T + t of `in`.  q and k are rotated
  * first: dimension i < rot_dims / 2 with i + rot_dims / 2 by table[pos0[s] + step + t][i] = (cos, sin); k is then multiplied
- * by k_scale.  decay: device fp32 [H]; state_in / state_out: device fp32 [n_seq, H, dim, vdim] (NULL: zeros / not wanted; the
+ * by k_scale.  decay: device fp32 [H], min_decay: the smallest of them (chooses the kernel); state_in / state_out: device fp32 [n_seq, H, dim, vdim] (NULL: zeros / not wanted; the
  * same pointer only for T = 1); y: [n_seq*T, H*vdim] in dtype; workspace from the _bytes call, 16-byte aligned.
  * impl: 0 = choose, 1 = recurrent, 2 = chunks on tcgen05 or fail.  status as elsewhere. */
 size_t dgpt_retention_workspace_bytes(int32_t n_seq, int32_t T, int32_t H, int32_t dim, int32_t vdim);
 int dgpt_retention(const void* in, int64_t in_row_stride, int32_t q_col, int32_t k_col, int32_t v_col, int32_t g_col,
                    const float* table, int32_t table_len, int32_t rot_dims, const int32_t* pos0, const int32_t* step_ptr,
-                   const float* decay, float k_scale, const float* state_in, float* state_out, float eps, void* y,
-                   int64_t y_row_stride, float* workspace, size_t workspace_bytes, int32_t n_seq, int32_t T, int32_t H,
+                   const float* decay, float min_decay, float k_scale, const float* state_in, float* state_out, float eps,
+                   void* y, int64_t y_row_stride, float* workspace, size_t workspace_bytes, int32_t n_seq, int32_t T, int32_t H,
                    int32_t dim, int32_t vdim, int32_t dtype, int32_t impl, int32_t* status, void* stream);
 
 #ifdef __cplusplus

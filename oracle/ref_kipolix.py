@@ -164,7 +164,7 @@ def forward(cfg: dict, w: dict, ids, keep_layers: bool = False):
 
 
 # ---- small random models for the tests -------------------------------------------------
-def random_model(cfg: dict, seed: int, std: float = 0.5) -> dict:
+def random_model(cfg: dict, seed: int, std: float = 0.4) -> dict:
     """Weights for a configuration, float32 but representable in bfloat16, so that both number formats start from the
     same numbers.  Norm weights scatter around 0 (1 for the query and key norms); the streams differ from the first
     sublayer on."""
@@ -196,6 +196,6 @@ def random_model(cfg: dict, seed: int, std: float = 0.5) -> dict:
             w[p + "norm2"] = near(0.0, C)
             w[p + "mlp.gate"], w[p + "mlp.up"], w[p + "mlp.down"] = lin(f, C), lin(f, C), lin(C, f)
         for q in subs:
-            w[f"{p}hc{q}.in"], w[f"{p}hc{q}.out"] = near(1.0 / S, S), near(0.8, S)
-            w[f"{p}hc{q}.mix"] = 0.8 * torch.eye(S) + 0.15 * torch.randn(S, S, generator=g)
+            w[f"{p}hc{q}.in"], w[f"{p}hc{q}.out"] = near(1.0 / S, S), 0.5 * near(0.8, S)
+            w[f"{p}hc{q}.mix"] = 0.9 * torch.eye(S) + 0.1 * torch.randn(S, S, generator=g)
     return {k: v.to(torch.bfloat16).float() for k, v in w.items()}
