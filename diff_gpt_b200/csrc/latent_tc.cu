@@ -106,49 +106,6 @@ __device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map
       ::"r"(dst), "l"(reinterpret_cast<uint64_t>(map)), "r"(bar), "r"(c0), "r"(c1), "r"(c2)
       : "memory");
 }
-__device__ __forceinline__ void tmem_ld16_nowait(uint32_t addr, float* v) {
-  uint32_t* r = reinterpret_cast<uint32_t*>(v);
-  asm volatile(
-      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
-      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
-      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
-        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
-      : "r"(addr)
-      : "memory");
-}
-// Eight MMAs over one unit in a single statement with constant descriptor steps.  Offsets in 16-byte units: A advances by
-// A_STEP, B by 2 (16 elements along its 128-byte rows); the second four start at A_HALF and B_HALF.  The first MMA takes
-// the accumulate flag.
-template <int A_STEP, int A_HALF, int B_HALF>
-__device__ __forceinline__ void lt_mma8(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
-  asm volatile(
-      "{\n\t.reg .pred p0, pt;\n\t.reg .b64 a, b;\n\t"
-      "setp.ne.b32 p0, %4, 0;\n\tsetp.eq.b32 pt, 0, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p0;\n\t"
-      "add.u64 a, %1, %5;\n\tadd.u64 b, %2, 2;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %6;\n\tadd.u64 b, %2, 4;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %7;\n\tadd.u64 b, %2, 6;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %8;\n\tadd.u64 b, %2, %12;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %9;\n\tadd.u64 b, %2, %13;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %10;\n\tadd.u64 b, %2, %14;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %11;\n\tadd.u64 b, %2, %15;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t}"
-      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP), "n"(A_HALF), "n"(A_HALF + A_STEP),
-      "n"(A_HALF + 2 * A_STEP), "n"(A_HALF + 3 * A_STEP), "n"(B_HALF), "n"(B_HALF + 2), "n"(B_HALF + 4), "n"(B_HALF + 6)
-      : "memory");
-}
-// The first four of those MMAs: a unit of one block.
-template <int A_STEP>
-__device__ __forceinline__ void lt_mma4(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
-  asm volatile(
-      "{\n\t.reg .pred p0, pt;\n\t.reg .b64 a, b;\n\t"
-      "setp.ne.b32 p0, %4, 0;\n\tsetp.eq.b32 pt, 0, 0;\n\t"
-      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p0;\n\t"
-      "add.u64 a, %1, %5;\n\tadd.u64 b, %2, 2;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %6;\n\tadd.u64 b, %2, 4;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
-      "add.u64 a, %1, %7;\n\tadd.u64 b, %2, 6;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t}"
-      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP)
-      : "memory");
-}
 // The four softmax warps: a barrier, and a barrier that tells every thread whether any of them said yes.
 __device__ __forceinline__ void lt_sync() { asm volatile("barrier.sync 1, 128;" ::: "memory"); }
 __device__ __forceinline__ bool lt_any(bool mine) {
@@ -310,8 +267,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
             if (!ok) return;
             tc_fence_after();
             const uint64_t da = dC + ((aU + s * unit_bytes) >> 4), db = dC + ((aQ + 2 * u * kQBlock) >> 4);
-            if (lt_blocks(p.a.dk, u) == 2) lt_mma8<2, kLtBlock / 16, kQBlock / 16>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
-            else lt_mma4<2>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
+            if (lt_blocks(p.a.dk, u) == 2) umma_ss8<2, kLtBlock / 16, 2, kQBlock / 16>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
+            else umma_ss4<2, 2>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
             if (!shared_kv) umma_commit(bar_uf + 8 * s);  // keys are done with
           }
           umma_commit(bar_s + 8 * (gt & 1u));
@@ -332,7 +289,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
               if (!ok) break;
               tc_fence_after();
             }
-            lt_mma8<128, 512, kPBlock / 16>(tmem + 2 * N + u * N, dM + ((aU + s * unit_bytes) >> 4), dC + ((aP + (ahead ? 2 * b * kPBlock : 0u)) >> 4),
+            umma_ss8<128, 512, 2, kPBlock / 16>(tmem + 2 * N + u * N, dM + ((aU + s * unit_bytes) >> 4), dC + ((aP + (ahead ? 2 * b * kPBlock : 0u)) >> 4),
                                             kIdescO, j > 0 ? 1u : 0u);
             umma_commit(bar_uf + 8 * s);
           }

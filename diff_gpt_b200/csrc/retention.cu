@@ -46,43 +46,54 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   float* so = sk + a.dim_pad;       // [groups][vdim]
   __shared__ float scratch[40];
   const int h = blockIdx.x % a.H, s = blockIdx.x / a.H, tid = threadIdx.x;
+  const int g = tid / cols, c = (tid - g * cols) * 4;
+  const bool work = g < groups;
+  const long long base = ((long long)s * a.H + h) * dim * e + c;
+  const float* in = a.state_in + base;
+  float* out = a.state_out + base;
+  // the first rows of the state are on their way while q and k are rotated
+  constexpr int U = 8;
+  float4 r[U];
+#pragma unroll
+  for (int u = 0; u < U; ++u)
+    if (work && g + u * groups < dim) r[u] = *reinterpret_cast<const float4*>(in + (long long)(g + u * groups) * e);
   const int pos = a.pos0[s] + (a.step_ptr ? *a.step_ptr : 0);
   const bool ok = pos >= 0 && pos < a.table_len;
   if (!ok && tid == 0 && a.status) *a.status = 1;
   const float2* cs = a.table + (long long)(ok ? pos : 0) * (a.rot >> 1);
   const T* row = static_cast<const T*>(a.in) + (long long)s * a.in_rs;
-  if (tid < 128) rotate_head<T>(row + a.q_col + h * dim, cs, a.rot, dim, 1.f, sq, tid, 128);
-  else rotate_head<T>(row + a.k_col + h * dim, cs, a.rot, dim, a.k_scale, sk, tid - 128, 128);
-  const int g = tid / cols, c = (tid - g * cols) * 4;
-  const bool work = g < groups;
   FVec<4> v;
   if (work) v = ldt<T, 4>(row + a.v_col + h * e + c);
+  const bool mine = tid < cols;
+  FVec<4> gv;
+  if (mine) gv = ldt<T, 4>(row + a.g_col + h * e + c);
+  if (tid < 128) rotate_head<T>(row + a.q_col + h * dim, cs, a.rot, dim, 1.f, sq, tid, 128);
+  else rotate_head<T>(row + a.k_col + h * dim, cs, a.rot, dim, a.k_scale, sk, tid - 128, 128);
   const float decay = a.decay[h];
   __syncthreads();
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
   if (work) {
-    const long long base = ((long long)s * a.H + h) * dim * e + c;
-    const float* in = a.state_in + base;
-    float* out = a.state_out + base;
-    for (int d = g; d < dim; d += 8 * groups) {
-      float4 r[8];
+    for (int d = g; d < dim; d += U * groups) {
+      float4 cur[U];
 #pragma unroll
-      for (int u = 0; u < 8; ++u)
-        if (d + u * groups < dim) r[u] = *reinterpret_cast<const float4*>(in + (long long)(d + u * groups) * e);
+      for (int u = 0; u < U; ++u) cur[u] = r[u];
 #pragma unroll
-      for (int u = 0; u < 8; ++u) {
+      for (int u = 0; u < U; ++u)
+        if (d + (U + u) * groups < dim) r[u] = *reinterpret_cast<const float4*>(in + (long long)(d + (U + u) * groups) * e);
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
         const int i = d + u * groups;
         if (i < dim) {
           const float kd = sk[i], qd = sq[i];
-          r[u].x = fmaf(decay, r[u].x, kd * v.v[0]);
-          r[u].y = fmaf(decay, r[u].y, kd * v.v[1]);
-          r[u].z = fmaf(decay, r[u].z, kd * v.v[2]);
-          r[u].w = fmaf(decay, r[u].w, kd * v.v[3]);
-          *reinterpret_cast<float4*>(out + (long long)i * e) = r[u];
-          acc[0] = fmaf(qd, r[u].x, acc[0]);
-          acc[1] = fmaf(qd, r[u].y, acc[1]);
-          acc[2] = fmaf(qd, r[u].z, acc[2]);
-          acc[3] = fmaf(qd, r[u].w, acc[3]);
+          cur[u].x = fmaf(decay, cur[u].x, kd * v.v[0]);
+          cur[u].y = fmaf(decay, cur[u].y, kd * v.v[1]);
+          cur[u].z = fmaf(decay, cur[u].z, kd * v.v[2]);
+          cur[u].w = fmaf(decay, cur[u].w, kd * v.v[3]);
+          *reinterpret_cast<float4*>(out + (long long)i * e) = cur[u];
+          acc[0] = fmaf(qd, cur[u].x, acc[0]);
+          acc[1] = fmaf(qd, cur[u].y, acc[1]);
+          acc[2] = fmaf(qd, cur[u].z, acc[2]);
+          acc[3] = fmaf(qd, cur[u].w, acc[3]);
         }
       }
     }
@@ -91,7 +102,6 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   __syncthreads();
   float o[4] = {0.f, 0.f, 0.f, 0.f};
   float ss = 0.f;
-  const bool mine = tid < cols;
   if (mine) {
     for (int i = 0; i < groups; ++i) {
       const float4 p = *reinterpret_cast<const float4*>(so + i * e + c);
@@ -104,7 +114,6 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   }
   const float inv = rsqrtf(block_sum(ss, scratch) / (float)e + a.eps);
   if (mine) {
-    const FVec<4> gv = ldt<T, 4>(row + a.g_col + h * e + c);
     FVec<4> y;
 #pragma unroll
     for (int i = 0; i < 4; ++i) y.v[i] = o[i] * inv * silu_value(gv.v[i]);

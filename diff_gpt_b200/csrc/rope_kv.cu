@@ -193,70 +193,166 @@ __device__ __forceinline__ void st4(T* p, const float* v) {
   Pair<T>::st(p + 2, v[2], v[3]);
 }
 
+// where the cache row of slot `slot` of sequence s lies, or NULL
+template <typename T>
+__device__ __forceinline__ T* cache_row(const KvView& kv, int s, int slot, int row_w) {
+  const int cap = kv.page_table ? kv.max_pages * kv.page_tokens : kv.page_tokens;
+  if (slot < 0 || slot >= cap) return nullptr;
+  const int lp = slot / kv.page_tokens;
+  long long pg = s;
+  if (kv.page_table) pg = kv.page_table[(long long)s * kv.max_pages + lp];
+  if (pg < 0 || (kv.n_pages > 0 && pg >= kv.n_pages)) return nullptr;
+  return static_cast<T*>(kv.k) + pg * kv.page_stride + (long long)(slot - lp * kv.page_tokens) * row_w;
+}
+
+struct ProjArgs {
+  long long in_rs, q_rs;
+  const float *qw, *kw;
+  float q_count, k_count, eps;
+  const float2* table;
+  int table_len, rot, row_w;
+  const int *pos0, *slot0, *step_ptr;
+  int Tn, HD, GD, GE, D;
+  int* status;
+};
+
+// One warp per token, q and k of the token in registers as they were loaded (NV 16-byte pieces per lane).
+template <typename T, int NV>
+__global__ void __launch_bounds__(256)
+proj_norm_rope_append_warp_kernel(const T* __restrict__ in, T* __restrict__ q_out, const KvView kv, const ProjArgs a, long long n_tok) {
+  constexpr int VEC = Io<T>::kVec16;
+  const long long tok = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  if (tok >= n_tok) return;
+  const int lane = threadIdx.x & 31;
+  const int s = (int)(tok / a.Tn), t = (int)(tok - (long long)s * a.Tn);
+  const T* row = in + tok * a.in_rs;
+  const int n = a.HD + a.GD;
+  uint4 raw[NV];
+  float qs = 0.f, ks = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (lane + 32 * i) * VEC;
+    raw[i] = make_uint4(0u, 0u, 0u, 0u);
+    if (c < n) raw[i] = __ldg(reinterpret_cast<const uint4*>(row + c));
+  }
+  const int step = a.step_ptr ? *a.step_ptr : 0;
+  const int pos = a.pos0[s] + step + t;
+  T* dst = cache_row<T>(kv, s, a.slot0[s] + step + t, a.row_w);
+  const bool ok = pos >= 0 && pos < a.table_len;
+  if ((dst == nullptr || !ok) && lane == 0 && a.status) *a.status = 1;
+  const float2* cs = a.table + (long long)(ok ? pos : 0) * (a.rot >> 1);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (lane + 32 * i) * VEC;
+    float v[VEC], ss = 0.f;
+    unpack16<T>(raw[i], v);
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) ss += v[e] * v[e];
+    if (c < a.HD) qs += ss;
+    else ks += ss;
+  }
+  const float qi = rsqrtf(warp_sum(qs) / a.q_count + a.eps), ki = rsqrtf(warp_sum(ks) / a.k_count + a.eps);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int c = (lane + 32 * i) * VEC;
+    if (c >= n) continue;
+    const bool is_q = c < a.HD;
+    const int x = is_q ? c : c - a.HD, d = x % a.D;
+    const float inv = is_q ? qi : ki;
+    const float* w = (is_q ? a.qw : a.kw) + x;
+    float v[VEC];
+    unpack16<T>(raw[i], v);
+#pragma unroll
+    for (int e = 0; e < VEC; e += 4) {
+      const float4 f = __ldg(reinterpret_cast<const float4*>(w + e));
+      v[e] *= inv * f.x; v[e + 1] *= inv * f.y; v[e + 2] *= inv * f.z; v[e + 3] *= inv * f.w;
+    }
+#pragma unroll
+    for (int e = 0; e < VEC; e += 2) {
+      if (d + e < a.rot) {
+        const float2 f = __ldg(cs + ((d + e) >> 1));
+        const float p = v[e], q = v[e + 1];
+        v[e] = p * f.x - q * f.y;
+        v[e + 1] = q * f.x + p * f.y;
+      }
+    }
+    if (is_q) st16<T>(q_out + tok * a.q_rs + x, v, 1.f);
+    else if (dst) st16<T>(dst + x, v, 1.f);
+  }
+  if (dst)
+    for (int c = lane * VEC; c < a.GE; c += 32 * VEC)
+      *reinterpret_cast<uint4*>(dst + a.GD + c) = __ldg(reinterpret_cast<const uint4*>(row + n + c));
+}
+
+// CTA per token, rows of any length.
 template <typename T>
 __global__ void __launch_bounds__(kRowsThreads)
-proj_norm_rope_append_kernel(const T* __restrict__ in, long long in_rs, const float* __restrict__ qw, const float* __restrict__ kw,
-                             float q_count, float k_count, float eps, const float2* __restrict__ table, int table_len, int rot,
-                             T* __restrict__ q_out, long long q_rs, KvView kv, int row_w, const int* __restrict__ pos0,
-                             const int* __restrict__ slot0, const int* __restrict__ step_ptr, int Tn, int HD, int GD, int GE, int D,
-                             int* status) {
+proj_norm_rope_append_kernel(const T* __restrict__ in, T* __restrict__ q_out, const KvView kv, const ProjArgs a) {
   __shared__ float scratch[40], scratch2[40];
   const long long tok = blockIdx.x;
-  const int s = (int)(tok / Tn), t = (int)(tok - (long long)s * Tn), tid = threadIdx.x;
-  const int step = step_ptr ? *step_ptr : 0;
-  const int pos = pos0[s] + step + t, slot = slot0[s] + step + t;
-  const int cap = kv.page_table ? kv.max_pages * kv.page_tokens : kv.page_tokens;
-  T* dst = nullptr;
-  if (slot >= 0 && slot < cap) {
-    const int lp = slot / kv.page_tokens;
-    long long pg = s;
-    if (kv.page_table) pg = kv.page_table[(long long)s * kv.max_pages + lp];
-    if (pg >= 0 && (kv.n_pages <= 0 || pg < kv.n_pages))
-      dst = static_cast<T*>(kv.k) + pg * kv.page_stride + (long long)(slot - lp * kv.page_tokens) * row_w;
-  }
-  const bool ok = pos >= 0 && pos < table_len;
-  if ((dst == nullptr || !ok) && tid == 0 && status) *status = 1;
-  const float2* cs = table + (long long)(ok ? pos : 0) * (rot >> 1);
-  const T* row = in + tok * in_rs;
-  const int n = HD + GD;
+  const int s = (int)(tok / a.Tn), t = (int)(tok - (long long)s * a.Tn), tid = threadIdx.x;
+  const int step = a.step_ptr ? *a.step_ptr : 0;
+  const int pos = a.pos0[s] + step + t;
+  T* dst = cache_row<T>(kv, s, a.slot0[s] + step + t, a.row_w);
+  const bool ok = pos >= 0 && pos < a.table_len;
+  if ((dst == nullptr || !ok) && tid == 0 && a.status) *a.status = 1;
+  const float2* cs = a.table + (long long)(ok ? pos : 0) * (a.rot >> 1);
+  const T* row = in + tok * a.in_rs;
+  const int n = a.HD + a.GD;
   float qs = 0.f, ks = 0.f;
   for (int c = tid * 4; c < n; c += kRowsThreads * 4) {
     float v[4];
     ld4<T>(row + c, v);
     const float ss = v[0] * v[0] + v[1] * v[1] + v[2] * v[2] + v[3] * v[3];
-    if (c < HD) qs += ss;
+    if (c < a.HD) qs += ss;
     else ks += ss;
   }
   qs = block_sum(qs, scratch);
   ks = block_sum(ks, scratch2);
-  const float qi = rsqrtf(qs / q_count + eps), ki = rsqrtf(ks / k_count + eps);
+  const float qi = rsqrtf(qs / a.q_count + a.eps), ki = rsqrtf(ks / a.k_count + a.eps);
   for (int c = tid * 4; c < n; c += kRowsThreads * 4) {
-    const bool is_q = c < HD;
-    const int x = is_q ? c : c - HD, d = x % D;
+    const bool is_q = c < a.HD;
+    const int x = is_q ? c : c - a.HD, d = x % a.D;
     float v[4];
     ld4<T>(row + c, v);  // in L1 from the first pass
-    const float4 w = *reinterpret_cast<const float4*>((is_q ? qw : kw) + x);
+    const float4 w = *reinterpret_cast<const float4*>((is_q ? a.qw : a.kw) + x);
     const float inv = is_q ? qi : ki;
     v[0] *= inv * w.x; v[1] *= inv * w.y; v[2] *= inv * w.z; v[3] *= inv * w.w;
 #pragma unroll
     for (int p = 0; p < 2; ++p) {
-      if (d + 2 * p < rot) {
+      if (d + 2 * p < a.rot) {
         const float2 f = cs[(d >> 1) + p];
-        const float a = v[2 * p], b = v[2 * p + 1];
-        v[2 * p] = a * f.x - b * f.y;
-        v[2 * p + 1] = b * f.x + a * f.y;
+        const float x0 = v[2 * p], x1 = v[2 * p + 1];
+        v[2 * p] = x0 * f.x - x1 * f.y;
+        v[2 * p + 1] = x1 * f.x + x0 * f.y;
       }
     }
-    if (is_q) st4<T>(q_out + tok * q_rs + x, v);
+    if (is_q) st4<T>(q_out + tok * a.q_rs + x, v);
     else if (dst) st4<T>(dst + x, v);
   }
   if (dst) {
-    for (int c = tid * 4; c < GE; c += kRowsThreads * 4) {
+    for (int c = tid * 4; c < a.GE; c += kRowsThreads * 4) {
       float v[4];
       ld4<T>(row + n + c, v);
-      st4<T>(dst + GD + c, v);
+      st4<T>(dst + a.GD + c, v);
     }
   }
+}
+
+template <typename T>
+static int proj_launch(const void* in, void* q_out, const KvView& view, const ProjArgs& a, long long n_tok, cudaStream_t st) {
+  const T* x = static_cast<const T*>(in);
+  T* q = static_cast<T*>(q_out);
+  const int nv = (a.HD + a.GD + 32 * Io<T>::kVec16 - 1) / (32 * Io<T>::kVec16);
+  const unsigned grid = (unsigned)((n_tok + 7) / 8);
+  if (n_tok < 148 * 8 || nv > 16) proj_norm_rope_append_kernel<T><<<(unsigned)n_tok, kRowsThreads, 0, st>>>(x, q, view, a);  // few tokens: a CTA each
+  else if (nv <= 2) proj_norm_rope_append_warp_kernel<T, 2><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  else if (nv <= 4) proj_norm_rope_append_warp_kernel<T, 4><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  else if (nv <= 6) proj_norm_rope_append_warp_kernel<T, 6><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  else if (nv <= 8) proj_norm_rope_append_warp_kernel<T, 8><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  else if (nv <= 12) proj_norm_rope_append_warp_kernel<T, 12><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  else proj_norm_rope_append_warp_kernel<T, 16><<<grid, 256, 0, st>>>(x, q, view, a, n_tok);
+  return launch_status("proj_norm_rope_append");
 }
 
 }  // namespace dgpt
@@ -343,18 +439,16 @@ extern "C" int dgpt_proj_norm_rope_append(const void* in, int64_t in_row_stride,
   const long long n = (long long)n_seq * T;
   if (n == 0) return DGPT_OK;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const KvView view = make_view(kv);
-#define DGPT_PR(TT)                                                                                                         \
-  proj_norm_rope_append_kernel<TT><<<(unsigned)n, kRowsThreads, 0, st>>>(                                                   \
-      static_cast<const TT*>(in), in_row_stride, q_weight, k_weight, (float)q_count, (float)k_count, eps,                   \
-      reinterpret_cast<const float2*>(table), table_len, rot_dims, static_cast<TT*>(q_out), q_out_row_stride, view, row_width, \
-      seq_pos0, seq_slot0, step_ptr, T, H * D, G * D, G * Dv, D, status)
-  if (dtype == DGPT_F32) DGPT_PR(float);
-  else if (dtype == DGPT_BF16) DGPT_PR(__nv_bfloat16);
-  else {
-    set_error("proj_norm_rope_append: unknown dtype %d", dtype);
-    return DGPT_E_UNSUPPORTED;
-  }
-#undef DGPT_PR
-  return launch_status("proj_norm_rope_append");
+  ProjArgs a;
+  a.in_rs = in_row_stride; a.q_rs = q_out_row_stride;
+  a.qw = q_weight; a.kw = k_weight;
+  a.q_count = (float)q_count; a.k_count = (float)k_count; a.eps = eps;
+  a.table = reinterpret_cast<const float2*>(table); a.table_len = table_len; a.rot = rot_dims; a.row_w = row_width;
+  a.pos0 = seq_pos0; a.slot0 = seq_slot0; a.step_ptr = step_ptr;
+  a.Tn = T; a.HD = H * D; a.GD = G * D; a.GE = G * Dv; a.D = D;
+  a.status = status;
+  if (dtype == DGPT_F32) return proj_launch<float>(in, q_out, make_view(kv), a, n, st);
+  if (dtype == DGPT_BF16) return proj_launch<__nv_bfloat16>(in, q_out, make_view(kv), a, n, st);
+  set_error("proj_norm_rope_append: unknown dtype %d", dtype);
+  return DGPT_E_UNSUPPORTED;
 }

@@ -38,13 +38,13 @@ __device__ __forceinline__ bool mbar_try_wait(uint32_t bar, uint32_t parity) {
 // not, and must stay out of the fast path).  4e9 cycles is about two seconds.
 constexpr long long kWaitLimitCycles = 4000000000ll;
 // Bounded wait: false if the phase did not complete within the limit.
-__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity) {
+__device__ __forceinline__ bool mbar_wait(uint32_t bar, uint32_t parity, long long limit_cycles = kWaitLimitCycles) {
   if (mbar_try_wait(bar, parity)) return true;
   const long long t0 = clock64();
   for (;;) {
     for (int i = 0; i < 32; ++i)
       if (mbar_try_wait(bar, parity)) return true;
-    if (clock64() - t0 > kWaitLimitCycles) return false;
+    if (clock64() - t0 > limit_cycles) return false;
   }
 }
 
@@ -121,6 +121,18 @@ __device__ __forceinline__ void tmem_ld32_nowait(uint32_t addr, float* v) {
         "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]),
         "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]),
         "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
+      : "r"(addr)
+      : "memory");
+}
+
+// 16 columns, the wait left to the caller
+__device__ __forceinline__ void tmem_ld16_nowait(uint32_t addr, float* v) {
+  uint32_t* r = reinterpret_cast<uint32_t*>(v);
+  asm volatile(
+      "tcgen05.ld.sync.aligned.32x32b.x16.b32 "
+      "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];"
+      : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]),
+        "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15])
       : "r"(addr)
       : "memory");
 }
@@ -292,6 +304,40 @@ __device__ __forceinline__ void umma_ts_chain(uint32_t d_tmem, uint32_t a_tmem, 
         ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc)
         : "memory");
   }
+}
+
+// Eight (four) MMAs with both operands in shared memory in a single statement with constant descriptor steps, in 16-byte
+// units: the operands advance by A_STEP and B_STEP, the second four MMAs start at A_HALF and B_HALF.  The first MMA takes the
+// accumulate flag.  (Written out one by one, the compiler keeps every descriptor of a loop in a register of its own.)
+template <int A_STEP, int A_HALF, int B_STEP, int B_HALF>
+__device__ __forceinline__ void umma_ss8(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p0, pt;\n\t.reg .b64 a, b;\n\t"
+      "setp.ne.b32 p0, %4, 0;\n\tsetp.eq.b32 pt, 0, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p0;\n\t"
+      "add.u64 a, %1, %5;\n\tadd.u64 b, %2, %12;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %6;\n\tadd.u64 b, %2, %13;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %7;\n\tadd.u64 b, %2, %14;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %8;\n\tadd.u64 b, %2, %15;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %9;\n\tadd.u64 b, %2, %16;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %10;\n\tadd.u64 b, %2, %17;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %11;\n\tadd.u64 b, %2, %18;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP), "n"(A_HALF), "n"(A_HALF + A_STEP),
+      "n"(A_HALF + 2 * A_STEP), "n"(A_HALF + 3 * A_STEP), "n"(B_STEP), "n"(2 * B_STEP), "n"(3 * B_STEP), "n"(B_HALF), "n"(B_HALF + B_STEP),
+      "n"(B_HALF + 2 * B_STEP), "n"(B_HALF + 3 * B_STEP)
+      : "memory");
+}
+template <int A_STEP, int B_STEP>
+__device__ __forceinline__ void umma_ss4(uint32_t d, uint64_t a, uint64_t b, uint32_t idesc, uint32_t acc) {
+  asm volatile(
+      "{\n\t.reg .pred p0, pt;\n\t.reg .b64 a, b;\n\t"
+      "setp.ne.b32 p0, %4, 0;\n\tsetp.eq.b32 pt, 0, 0;\n\t"
+      "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p0;\n\t"
+      "add.u64 a, %1, %5;\n\tadd.u64 b, %2, %8;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %6;\n\tadd.u64 b, %2, %9;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t"
+      "add.u64 a, %1, %7;\n\tadd.u64 b, %2, %10;\n\ttcgen05.mma.cta_group::1.kind::f16 [%0], a, b, %3, pt;\n\t}"
+      ::"r"(d), "l"(a), "l"(b), "r"(idesc), "r"(acc), "n"(A_STEP), "n"(2 * A_STEP), "n"(3 * A_STEP), "n"(B_STEP), "n"(2 * B_STEP), "n"(3 * B_STEP)
+      : "memory");
 }
 
 constexpr int kBM = 128;  // query rows per MMA (the M of every tcgen05.mma here)

@@ -138,9 +138,14 @@ def test_silu_gate_alone_and_in_the_gemm(dtype):
 def test_projection_norm_rotation_and_append(dtype, H, G, dim, vdim, D, rot, base):
     """Norm over all heads at once, interleaved pairs on the leading dimensions, rows through a page table and in a dense
     run, positions that differ from slots, padding columns that do not count."""
+    for T in (37, 640):  # a CTA per token, a warp per token
+        check_append(dtype, H, G, dim, vdim, D, rot, base, T)
+
+
+def check_append(dtype, H, G, dim, vdim, D, rot, base, T):
     from diff_gpt_b200 import ops
 
-    g, B, T, pt, eps, pos0, slot0 = gen(H * D), 2, 37, 16, 1e-4, [900, 3], [5, 11]
+    g, B, pt, eps, pos0, slot0 = gen(H * D), 2, 16, 1e-4, [300, 3], [5, 11]
     q, k, v = rnd(g, B, T, H, dim, dtype=dtype), rnd(g, B, T, G, dim, dtype=dtype), rnd(g, B, T, G, vdim, dtype=dtype)
     qw, kw = rnd(g, H, dim), rnd(g, G, dim)
 
@@ -149,8 +154,9 @@ def test_projection_norm_rotation_and_append(dtype, H, G, dim, vdim, D, rot, bas
 
     x = torch.cat([pad(q, D), pad(k, D), pad(v, D), torch.full((B, T, 8), 9.0).to(dtype)], dim=-1).reshape(B * T, -1).cuda()
     W = 2 * G * D
-    n_pages = 11
-    perm = torch.randperm(n_pages, generator=g).int()[:10].view(2, 5)
+    per = -(-(T + 11) // pt)
+    n_pages = 2 * per + 1
+    perm = torch.randperm(n_pages, generator=g).int()[: 2 * per].view(2, per)
     pool = torch.full((n_pages, pt, W + 8), float("nan"), dtype=dtype, device="cuda")
     want_q = torch.stack([ref.rotate_pairs((ref.unit_rms(q[b].double().flatten(1), eps) * qw.double().flatten()).view(T, H, dim), rot, base, pos0[b])
                           for b in range(B)])
@@ -159,9 +165,9 @@ def test_projection_norm_rotation_and_append(dtype, H, G, dim, vdim, D, rot, bas
     step = torch.tensor([2], dtype=torch.int32, device="cuda")
     tab = table(base, rot, 1024)
     for paged in (True, False):
-        dense = torch.full((B, 64, W + 8), float("nan"), dtype=dtype, device="cuda")
+        dense = torch.full((B, T + 20, W + 8), float("nan"), dtype=dtype, device="cuda")
         lay = (ops.kv_layout(pool, pool, pool.stride(0), 0, pt, perm.cuda(), n_pages) if paged
-               else ops.kv_layout(dense, dense, dense.stride(0), 0, 64))
+               else ops.kv_layout(dense, dense, dense.stride(0), 0, T + 20))
         out = torch.empty(B * T, H * D, dtype=dtype, device="cuda")
         st = torch.zeros(1, dtype=torch.int32, device="cuda")
         ops.proj_norm_rope_append(
@@ -174,14 +180,13 @@ def test_projection_norm_rotation_and_append(dtype, H, G, dim, vdim, D, rot, bas
         close(got[..., :dim], want_q, dtype, bf16=6e-3)
         assert bool((got[..., dim:] == 0).all())
         for b in range(B):
-            for t in range(T):
-                s = slot0[b] + t
-                row = pool[perm[b, s // pt], s % pt] if paged else dense[b, s]
-                kr, vr = row[: G * D].view(G, D), row[G * D : W].view(G, D)
-                close(kr[:, :dim], want_k[b, t], dtype, f32=5e-5, bf16=8e-3)
-                assert torch.equal(vr[:, :vdim].cpu(), v[b, t]) and bool((kr[:, dim:] == 0).all()) and bool((vr[:, vdim:] == 0).all())
+            s = slot0[b] + torch.arange(T)
+            row = (pool[perm[b].long()[s // pt].cuda(), (s % pt).cuda()] if paged else dense[b, s.cuda()]).cpu()
+            kr, vr = row[:, : G * D].view(T, G, D), row[:, G * D : W].view(T, G, D)
+            close(kr[..., :dim], want_k[b], dtype, f32=5e-5, bf16=8e-3)
+            assert torch.equal(vr[..., :vdim], v[b]) and bool((kr[..., dim:] == 0).all()) and bool((vr[..., vdim:] == 0).all())
     ops.proj_norm_rope_append(x, pad(qw, D).cuda(), pad(kw, D).cuda(), H * dim, G * dim, eps, tab, out, lay, W + 8,
-                              torch.tensor([0, 1000], dtype=torch.int32).cuda(), torch.tensor([40, 0], dtype=torch.int32).cuda(), None,
+                              torch.tensor([0, 1000], dtype=torch.int32).cuda(), torch.tensor([T, 0], dtype=torch.int32).cuda(), None,
                               n_seq=B, T=T, H=H, G=G, D=D, Dv=D, status=st)
     assert int(st.item()) == 1  # a slot past the run, a position past the table: reported, nothing written there
 
