@@ -65,8 +65,6 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   FVec<4> v;
   if (work) v = ldt<T, 4>(row + a.v_col + h * e + c);
   const bool mine = tid < cols;
-  FVec<4> gv;
-  if (mine) gv = ldt<T, 4>(row + a.g_col + h * e + c);
   if (tid < 128) rotate_head<T>(row + a.q_col + h * dim, cs, a.rot, dim, 1.f, sq, tid, 128);
   else rotate_head<T>(row + a.k_col + h * dim, cs, a.rot, dim, a.k_scale, sk, tid - 128, 128);
   const float decay = a.decay[h];
@@ -74,26 +72,25 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   float acc[4] = {0.f, 0.f, 0.f, 0.f};
   if (work) {
     for (int d = g; d < dim; d += U * groups) {
-      float4 cur[U];
+      if (d != g) {
 #pragma unroll
-      for (int u = 0; u < U; ++u) cur[u] = r[u];
-#pragma unroll
-      for (int u = 0; u < U; ++u)
-        if (d + (U + u) * groups < dim) r[u] = *reinterpret_cast<const float4*>(in + (long long)(d + (U + u) * groups) * e);
+        for (int u = 0; u < U; ++u)
+          if (d + u * groups < dim) r[u] = *reinterpret_cast<const float4*>(in + (long long)(d + u * groups) * e);
+      }
 #pragma unroll
       for (int u = 0; u < U; ++u) {
         const int i = d + u * groups;
         if (i < dim) {
           const float kd = sk[i], qd = sq[i];
-          cur[u].x = fmaf(decay, cur[u].x, kd * v.v[0]);
-          cur[u].y = fmaf(decay, cur[u].y, kd * v.v[1]);
-          cur[u].z = fmaf(decay, cur[u].z, kd * v.v[2]);
-          cur[u].w = fmaf(decay, cur[u].w, kd * v.v[3]);
-          *reinterpret_cast<float4*>(out + (long long)i * e) = cur[u];
-          acc[0] = fmaf(qd, cur[u].x, acc[0]);
-          acc[1] = fmaf(qd, cur[u].y, acc[1]);
-          acc[2] = fmaf(qd, cur[u].z, acc[2]);
-          acc[3] = fmaf(qd, cur[u].w, acc[3]);
+          r[u].x = fmaf(decay, r[u].x, kd * v.v[0]);
+          r[u].y = fmaf(decay, r[u].y, kd * v.v[1]);
+          r[u].z = fmaf(decay, r[u].z, kd * v.v[2]);
+          r[u].w = fmaf(decay, r[u].w, kd * v.v[3]);
+          *reinterpret_cast<float4*>(out + (long long)i * e) = r[u];
+          acc[0] = fmaf(qd, r[u].x, acc[0]);
+          acc[1] = fmaf(qd, r[u].y, acc[1]);
+          acc[2] = fmaf(qd, r[u].z, acc[2]);
+          acc[3] = fmaf(qd, r[u].w, acc[3]);
         }
       }
     }
@@ -114,6 +111,7 @@ __global__ void __launch_bounds__(kRetThreads) retention_decode_kernel(const Ret
   }
   const float inv = rsqrtf(block_sum(ss, scratch) / (float)e + a.eps);
   if (mine) {
+    const FVec<4> gv = ldt<T, 4>(row + a.g_col + h * e + c);
     FVec<4> y;
 #pragma unroll
     for (int i = 0; i < 4; ++i) y.v[i] = o[i] * inv * silu_value(gv.v[i]);
