@@ -69,7 +69,10 @@ __device__ __forceinline__ int window_first_tile(int window, int first_q, int ti
 __device__ __forceinline__ int kept_tiles(int keep_first, int tile0, int tile) {
   return min(tile0, (keep_first + tile - 1) / tile);
 }
-__device__ __forceinline__ int tile_of(int j, int n_kept, int tile0) { return j < n_kept ? j : tile0 + (j - n_kept); }
+template <bool KEPT>
+__device__ __forceinline__ int tile_of(int j, int n_kept, int tile0) {
+  return KEPT && j < n_kept ? j : tile0 + (j - n_kept);
+}
 
 // warp-level kernel (fmha_simt.cu)
 int fmha_simt(const FmhaArgs& a, const KvView& kv, cudaStream_t st);

@@ -61,7 +61,7 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
 
   const int tile0 = window_first_tile(window, q_offset + q0, kSimtBN), n_kept = kept_tiles(keep_first, tile0, kSimtBN);
   for (int tile = 0;; ++tile) {
-    const int j0 = tile_of(tile, n_kept, tile0) * kSimtBN;
+    const int j0 = tile_of<true>(tile, n_kept, tile0) * kSimtBN;
     if (j0 >= kmax) break;
     __syncthreads();
     constexpr int VPR = D / VEC;  // 16-byte vectors per key row

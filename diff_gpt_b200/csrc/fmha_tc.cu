@@ -22,7 +22,7 @@ namespace tc {
 constexpr int kTmemCols = 256;    // S/P: [0,128), O tile: [128, 128 + D)
 
 
-template <int D>
+template <int D, bool KEPT>
 __global__ void __launch_bounds__(128, 2)
 fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk,
                const __grid_constant__ CUtensorMap mv, const TcParams p) {
@@ -92,12 +92,12 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
   const int klen = p.kv_len ? p.kv_len[b] : p.kv_len_all;
   const int kmax = p.causal ? min(klen, p.q_offset + min(q0 + kBM, p.Tq)) : klen;
   const int tile0 = window_first_tile(p.window, p.q_offset + q0, kBN);
-  const int n_kept = kept_tiles(p.keep_first, tile0, kBN), kvh = h / p.kv_div;
+  const int n_kept = KEPT ? kept_tiles(p.keep_first, tile0, kBN) : 0, kvh = p.kv_div == 1 ? h : h / p.kv_div;
   const int n_tiles = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0) + n_kept;
 
   // Issue the TMA loads of key/value tile j (thread 0 only).  One box per page and per 64-wide half.
   auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t bar, int j) {
-    const int t0 = tile_of(j, n_kept, tile0) * kBN;
+    const int t0 = tile_of<KEPT>(j, n_kept, tile0) * kBN;
     if (pt >= kBN) {
       const int lp = t0 / pt, in = t0 - lp * pt;
       const int pg = p.page_table ? p.page_table[(long long)b * p.max_pages + lp] : b;
@@ -131,7 +131,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
 
   for (int j = 0; j < n_tiles; ++j) {
     const uint32_t par = (uint32_t)(j & 1);
-    const int t0 = tile_of(j, n_kept, tile0) * kBN;
+    const int t0 = tile_of<KEPT>(j, n_kept, tile0) * kBN;
     // ---- S = Q K^T ----
     if (tid == 0) {
       bool ok = true;
@@ -186,7 +186,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
     if (need_mask) {
 #pragma unroll
       for (int i = 0; i < kBN; ++i) {
-        sv[i] = (t0 + i <= last_key && (t0 + i >= first_key || t0 + i < p.keep_first)) ? sv[i] : -INFINITY;
+        sv[i] = (t0 + i <= last_key && (t0 + i >= first_key || (KEPT && t0 + i < p.keep_first))) ? sv[i] : -INFINITY;
         mx = fmaxf(mx, sv[i]);
       }
     } else {
@@ -394,13 +394,17 @@ int fmha_tc(const FmhaArgs& a, const dgpt_kv_layout& kv, cudaStream_t st) {
   }
   // one CTA per work item, or fewer CTAs that loop over the items when the caller wants the kernel on few SMs
   const unsigned n_cta = (a.max_ctas > 0 && a.max_ctas < p.n_work) ? (unsigned)a.max_ctas : (unsigned)p.n_work;
-  if (D == 64) {
-    e = cudaFuncSetAttribute(fmha_tc_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) fmha_tc_kernel<64><<<n_cta, 128, smem, st>>>(mq, mk, mv, p);
-  } else {
-    e = cudaFuncSetAttribute(fmha_tc_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) fmha_tc_kernel<128><<<n_cta, 128, smem, st>>>(mq, mk, mv, p);
-  }
+#define DGPT_TC(DD, KK)                                                                                           \
+  do {                                                                                                            \
+    e = cudaFuncSetAttribute(fmha_tc_kernel<DD, KK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+    if (e == cudaSuccess) fmha_tc_kernel<DD, KK><<<n_cta, 128, smem, st>>>(mq, mk, mv, p);                        \
+  } while (0)
+  const bool kept = p.keep_first > 0;
+  if (D == 64 && kept) DGPT_TC(64, true);
+  else if (D == 64) DGPT_TC(64, false);
+  else if (kept) DGPT_TC(128, true);
+  else DGPT_TC(128, false);
+#undef DGPT_TC
   if (e != cudaSuccess) {
     set_error("fmha_tc: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     return DGPT_E_CUDA;

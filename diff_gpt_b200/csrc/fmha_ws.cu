@@ -35,23 +35,26 @@ constexpr int kWsThreads = 320;  // 8 softmax warps, the MMA issuer's warp, the 
 constexpr uint32_t kWsTmemCols = 512;
 
 struct WsItem {
-  int b, h, q0, klen, tile0, n_kept, n;  // n = key tiles: n_kept of kept first keys, then those from tile0 on (see tile_of)
+  int b, h, kvh, q0, klen, tile0, n_kept, n;  // n = key tiles: n_kept of kept first keys, then those from tile0 on (see tile_of)
 };
 
+template <bool KEPT>
 __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
   WsItem it;
   it.h = bh % p.H;
   it.b = bh / p.H;
+  it.kvh = p.kv_div == 1 ? it.h : it.h / p.kv_div;
   it.q0 = qt * kBM;
   it.klen = p.kv_len ? p.kv_len[it.b] : p.kv_len_all;
   const int kmax = p.causal ? min(it.klen, p.q_offset + min(it.q0 + kBM, p.Tq)) : it.klen;
   it.tile0 = window_first_tile(p.window, p.q_offset + it.q0, kBN);
-  it.n_kept = kept_tiles(p.keep_first, it.tile0, kBN);
+  it.n_kept = KEPT ? kept_tiles(p.keep_first, it.tile0, kBN) : 0;
   it.n = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0) + it.n_kept;
   return it;
 }
 
-template <int D>
+// KEPT: keys below p.keep_first are seen whatever the window (without it the kernel carries none of that)
+template <int D, bool KEPT>
 __global__ void __launch_bounds__(kWsThreads, 1)
 fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mk,
                   const __grid_constant__ CUtensorMap mv, const TcParams p) {
@@ -117,10 +120,10 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       unsigned kn = 0u, vn = 0u;    // K and V tiles whose loads have been issued (over all items)
       bool ok = true;
       while (ok && sched.next(bh, qt)) {
-        const WsItem it = ws_item(p, bh, qt);
+        const WsItem it = ws_item<KEPT>(p, bh, qt);
         if (it.n == 0) continue;
         auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t full, int j) {
-          const int t0 = tile_of(j, it.n_kept, it.tile0) * kBN, kvh = it.h / p.kv_div;
+          const int t0 = tile_of<KEPT>(j, it.n_kept, it.tile0) * kBN, kvh = it.kvh;
           if (pt >= kBN) {
             const int lp = t0 / pt, in = t0 - lp * pt;
             const int pg = p.page_table ? p.page_table[(long long)it.b * p.max_pages + lp] : it.b;
@@ -184,7 +187,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       unsigned items = 0u, g0 = 0u;
       bool ok = true;
       while (ok && sched.next(bh, qt)) {
-        const WsItem it = ws_item(p, bh, qt);
+        const WsItem it = ws_item<KEPT>(p, bh, qt);
         const int n = it.n;
         if (n == 0) continue;
         auto issue_s = [&](unsigned g, bool last) {  // S(g & 1) = Q K(g % 3)^T
@@ -261,12 +264,12 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       return collect(ok);
     };
     while (!fail && sched.next(bh, qt)) {
-      const WsItem it = ws_item(p, bh, qt);
+      const WsItem it = ws_item<KEPT>(p, bh, qt);
       const int n_tiles = it.n, klen = it.klen, q0 = it.q0, b = it.b, h = it.h;
       float m = -INFINITY, l = 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const unsigned g = g0 + (unsigned)j, buf = g & 1u, ph = (g >> 1) & 1u;
-        const int t0 = tile_of(j, it.n_kept, it.tile0) * kBN;
+        const int t0 = tile_of<KEPT>(j, it.n_kept, it.tile0) * kBN;
         // exits are taken by whole warps (the vote makes the decision uniform), never by single lanes
         if (!__all_sync(0xffffffffu, wait_or_abort(bar_s0 + 8 * buf, ph, abort_flag, 23))) {
           fail = true;
@@ -300,7 +303,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         tc_wait_ld();
         if (need_mask) {
 #pragma unroll
-          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key && (c0 + i >= first_key || c0 + i < p.keep_first)) ? sv[i] : -INFINITY;
+          for (int i = 0; i < kHalf; ++i) sv[i] = (c0 + i <= last_key && (c0 + i >= first_key || (KEPT && c0 + i < p.keep_first))) ? sv[i] : -INFINITY;
         }
         // One sweep turns this thread's 64 scores into probabilities against a reference maximum `ref` (log2 domain),
         // writes them as packed bf16 into the P buffer and returns their sum.
@@ -463,13 +466,17 @@ int fmha_tc_ws_launch(const FmhaArgs& a, const TcMaps& maps, TcParams p, long lo
   size_t smem = (size_t)6 * (D / 64) * kBN * 128 + 8192 + 1024;
   if (smem < 120 * 1024) smem = 120 * 1024;
   cudaError_t e;
-  if (D == 64) {
-    e = cudaFuncSetAttribute(fmha_tc_ws_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) fmha_tc_ws_kernel<64><<<n_cta, kWsThreads, smem, st>>>(maps.q, maps.k, maps.v, p);
-  } else {
-    e = cudaFuncSetAttribute(fmha_tc_ws_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    if (e == cudaSuccess) fmha_tc_ws_kernel<128><<<n_cta, kWsThreads, smem, st>>>(maps.q, maps.k, maps.v, p);
-  }
+#define DGPT_WS(DD, KK)                                                                                                          \
+  do {                                                                                                                           \
+    e = cudaFuncSetAttribute(fmha_tc_ws_kernel<DD, KK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                 \
+    if (e == cudaSuccess) fmha_tc_ws_kernel<DD, KK><<<n_cta, kWsThreads, smem, st>>>(maps.q, maps.k, maps.v, p);                 \
+  } while (0)
+  const bool kept = p.keep_first > 0;
+  if (D == 64 && kept) DGPT_WS(64, true);
+  else if (D == 64) DGPT_WS(64, false);
+  else if (kept) DGPT_WS(128, true);
+  else DGPT_WS(128, false);
+#undef DGPT_WS
   if (e != cudaSuccess) {
     set_error("fmha_tc: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     return DGPT_E_CUDA;

@@ -52,44 +52,58 @@ struct LtItem {
   int t0, n;                      // this split's tiles
 };
 
+// KEPT: the cache holds first keys that are seen from every distance, a slot range of their own
+template <bool KEPT>
 __device__ __forceinline__ LtItem lt_item(const LtParams& p, int item, int N) {
   LtItem it;
-  it.row = item % p.n_rows;
   const int gs = item / p.n_rows;
-  const int grp = gs % p.n_groups;
-  it.g = grp / p.gpk;
-  const int first = (grp - it.g * p.gpk) * N;
-  it.h0 = it.g * p.per + first;
+  it.row = item - gs * p.n_rows;
+  it.g = 0;
+  it.h0 = 0;
+  it.split = gs;
+  int first = 0;
+  if (p.n_groups > 1) {
+    it.split = gs / p.n_groups;
+    const int grp = gs - it.split * p.n_groups;
+    it.g = grp / p.gpk;
+    first = (grp - it.g * p.gpk) * N;
+    it.h0 = it.g * p.per + first;
+  }
   it.nh = min(N, p.per - first);
-  it.split = gs / p.n_groups;
   const LatentKeys k = latent_keys(p.a, it.row);
   it.seq = k.seq;
   // [0, ks) and [lo, n), cut where slots change from the first run to the second; the cut lies in one of the two
   const bool own = k.lo >= k.n0;
   it.begin[0] = 0;
-  it.end[0] = min(k.ks, k.n0);
+  it.end[0] = KEPT ? min(k.ks, k.n0) : 0;
   it.begin[1] = own ? k.s1 : k.lo;
-  it.end[1] = own ? k.s1 + max(0, k.ks - k.n0) : k.n0;
+  it.end[1] = own ? (KEPT ? k.s1 + max(0, k.ks - k.n0) : k.s1) : k.n0;
   it.begin[2] = k.s1 + max(0, k.lo - k.n0);
   it.end[2] = k.s1 + (k.n - k.n0);
   int nt[3];
 #pragma unroll
   for (int i = 0; i < 3; ++i) {
-    it.base[i] = it.begin[i] / p.align * p.align;
+    it.base[i] = it.begin[i] & ~(p.align - 1);  // a power of two
     nt[i] = it.end[i] > it.begin[i] ? (it.end[i] - it.base[i] + kLtKeys - 1) / kLtKeys : 0;
   }
-  it.n_first = nt[0];
-  it.n_second = nt[0] + nt[1];
+  it.n_first = KEPT ? nt[0] : 0;
+  it.n_second = it.n_first + nt[1];
   const int total = it.n_second + nt[2];
-  const int per = (total + p.a.n_splits - 1) / p.a.n_splits;
-  it.t0 = min(total, it.split * per);
-  it.n = min(total, it.t0 + per) - it.t0;
+  if (p.a.n_splits == 1) {
+    it.t0 = 0;
+    it.n = total;
+  } else {
+    const int per = (total + p.a.n_splits - 1) / p.a.n_splits;
+    it.t0 = min(total, it.split * per);
+    it.n = min(total, it.t0 + per) - it.t0;
+  }
   return it;
 }
 // first slot of tile j of the item, and the limits of its range
+template <bool KEPT>
 __device__ __forceinline__ int lt_tile(const LtItem& it, int j, int& begin, int& end) {
   const int t = it.t0 + j;
-  if (t < it.n_first) {
+  if (KEPT && t < it.n_first) {
     begin = it.begin[0];
     end = it.end[0];
     return it.base[0] + t * kLtKeys;
@@ -146,8 +160,9 @@ __device__ __forceinline__ float lt_reduce16(const float* v, int lane, F op) {
   return op(d, __shfl_xor_sync(0xffffffffu, d, 16));
 }
 
-// NB: heads per group = 16 NB; HS <= 16 NB: heads the softmax looks after (a group may hold fewer than 16)
-template <int NB, int HS>
+// NB: heads per group = 16 NB; HS <= 16 NB: heads the softmax looks after (a group may hold fewer than 16).
+// SHARED: a tile's values are its keys (latents), whose cache has no kept first keys.
+template <int NB, int HS, bool SHARED>
 __global__ void __launch_bounds__(kLtThreads, NB == 4 ? 1 : 2)
 latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ CUtensorMap mc, const LtParams p) {
   constexpr int N = 16 * NB;
@@ -159,10 +174,9 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int UT = p.upt, UK = p.uk, UV = p.uv, NU = p.n_units;
-  const bool shared_kv = p.a.v_col == 0;  // a tile's values are its keys
-  const int v_unit = shared_kv ? 0 : UK;  // where a tile's value units start
-  const int nqb = (p.a.dk + 63) / 64;     // 64-column blocks of Q
-  const uint32_t unit_bytes = p.unit_bytes;
+  const int v_unit = SHARED ? 0 : UK;  // where a tile's value units start
+  const int nqb = SHARED ? 2 * UK : (p.a.dk + 63) / 64;  // 64-column blocks of Q
+  const uint32_t unit_bytes = SHARED ? kLtUnit : p.unit_bytes;
   uint8_t* sU = smem;
   uint8_t* sQ = sU + (size_t)NU * unit_bytes;
   uint8_t* sP = sQ + (size_t)2 * UK * kQBlock;  // one or two buffers of two blocks
@@ -208,7 +222,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       const int pt = p.a.kv.page_tokens;
       const LatentArgs& a = p.a;
       for (int item = blockIdx.x; ok && item < p.n_items; item += gridDim.x) {
-        const LtItem it = lt_item(p, item, N);
+        const LtItem it = lt_item<!SHARED>(p, item, N);
         if (it.n == 0) continue;
         if (items > 0) ok = wait_or_abort(bar_qf, (items - 1) & 1u, abort_flag, 50);  // the last scores of the item before are done
         if (!ok) break;
@@ -217,7 +231,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         ++items;
         for (int j = 0; ok && j < it.n; ++j) {
           int begin, end;
-          const int slot = lt_tile(it, j, begin, end);
+          const int slot = lt_tile<!SHARED>(it, j, begin, end);
           const int boxes = min(kLtKeys / p.box, (end - slot + p.box - 1) / p.box);
           for (int u = 0; ok && u < UT; ++u, ++un) {
             const unsigned s = un % (unsigned)NU, round = un / (unsigned)NU;
@@ -225,8 +239,8 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
             if (!ok) break;
             const uint32_t full = bar_u + 8 * s, dst = aU + s * unit_bytes;
             const bool key = u < UK;
-            const int blocks = key ? lt_blocks(a.dk, u) : lt_blocks(a.dv, u - UK);
-            const int col = key ? it.g * a.dk + u * 128 : a.v_col + it.g * a.dv + (u - UK) * 128;
+            const int blocks = SHARED ? 2 : key ? lt_blocks(a.dk, u) : lt_blocks(a.dv, u - UK);
+            const int col = SHARED ? u * 128 : key ? it.g * a.dk + u * 128 : a.v_col + it.g * a.dv + (u - UK) * 128;
             mbar_expect_tx(full, (uint32_t)boxes * p.box * 128u * blocks);
             for (int b = 0; b < boxes; ++b) {
               const int at = slot + b * p.box;
@@ -256,7 +270,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       unsigned g = 0u, items = 0u;  // tiles; items
       bool ok = true;
       for (int item = blockIdx.x; ok && item < p.n_items; item += gridDim.x) {
-        const LtItem it = lt_item(p, item, N);
+        const LtItem it = lt_item<!SHARED>(p, item, N);
         if (it.n == 0) continue;
         ok = wait_or_abort(bar_q, items & 1u, abort_flag, 52);
         auto issue_s = [&](unsigned gt, bool last) {
@@ -267,9 +281,9 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
             if (!ok) return;
             tc_fence_after();
             const uint64_t da = dC + ((aU + s * unit_bytes) >> 4), db = dC + ((aQ + 2 * u * kQBlock) >> 4);
-            if (lt_blocks(p.a.dk, u) == 2) umma_ss8<2, kLtBlock / 16, 2, kQBlock / 16>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
+            if (SHARED || lt_blocks(p.a.dk, u) == 2) umma_ss8<2, kLtBlock / 16, 2, kQBlock / 16>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
             else umma_ss4<2, 2>(d, da, db, kIdescS, u > 0 ? 1u : 0u);
-            if (!shared_kv) umma_commit(bar_uf + 8 * s);  // keys are done with
+            if (!SHARED) umma_commit(bar_uf + 8 * s);  // keys are done with
           }
           umma_commit(bar_s + 8 * (gt & 1u));
           if (last) umma_commit(bar_qf);
@@ -284,7 +298,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
           tc_fence_after();
           for (int u = 0; u < UV; ++u) {
             const unsigned un = g * (unsigned)UT + (unsigned)(v_unit + u), s = un % (unsigned)NU;
-            if (!shared_kv) {
+            if (!SHARED) {
               ok = wait_or_abort(bar_u + 8 * s, (un / (unsigned)NU) & 1u, abort_flag, 53);
               if (!ok) break;
               tc_fence_after();
@@ -316,7 +330,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       lt_sync();
     }
     for (int item = blockIdx.x; item < p.n_items; item += gridDim.x) {
-      const LtItem it = lt_item(p, item, N);
+      const LtItem it = lt_item<!SHARED>(p, item, N);
       const int nh = it.nh;
       constexpr int HL = (N + 31) / 32;  // heads a lane looks after at the end of the item
       float gate[HL];
@@ -336,7 +350,7 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
       for (int j = 0; j < it.n; ++j, ++g) {
         const unsigned b = g & 1u;
         int begin, end;
-        const int slot = lt_tile(it, j, begin, end) + tid;
+        const int slot = lt_tile<!SHARED>(it, j, begin, end) + tid;
         if (!fail && !wait_or_abort(bar_s + 8 * b, (g >> 1) & 1u, abort_flag, 56)) fail = true;
         fail = __any_sync(0xffffffffu, fail);
         tc_fence_after();
@@ -344,9 +358,9 @@ latent_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__
         if (!fail && slot >= end) {  // nothing was loaded here, or rows nobody has written: 0 * x must stay 0
           for (int u = 0; u < UV; ++u) {
             const unsigned un = g * (unsigned)UT + (unsigned)(v_unit + u), us = un % (unsigned)NU;
-            if (!shared_kv && !wait_or_abort(bar_u + 8 * us, (un / (unsigned)NU) & 1u, abort_flag, 59)) break;  // still on its way
+            if (!SHARED && !wait_or_abort(bar_u + 8 * us, (un / (unsigned)NU) & 1u, abort_flag, 59)) break;  // still on its way
             uint8_t* unit = sU + (size_t)us * unit_bytes;
-            const bool two = lt_blocks(p.a.dv, u) == 2;
+            const bool two = SHARED || lt_blocks(p.a.dv, u) == 2;
 #pragma unroll
             for (int c = 0; c < 8; ++c) {
               reinterpret_cast<uint4*>(unit + tid * 128)[c] = make_uint4(0u, 0u, 0u, 0u);
@@ -537,18 +551,18 @@ static LtShape lt_shape(const LatentArgs& a) {
   s.uk = (a.dk + 127) / 128;
   s.uv = (a.dv + 127) / 128;
   s.upt = a.v_col == 0 ? s.uk : s.uk + s.uv;
-  s.unit_bytes = a.dk <= 64 && a.dv <= 64 ? kLtBlock : kLtUnit;
+  s.unit_bytes = a.v_col != 0 && a.dk <= 64 && a.dv <= 64 ? kLtBlock : kLtUnit;
   return s;
 }
 
-template <int NB, int HS>
+template <int NB, int HS, bool SHARED>
 static int lt_launch(const CUtensorMap& mq, const CUtensorMap& mc, const LtParams& p, int grid, size_t smem, cudaStream_t st) {
-  cudaError_t e = cudaFuncSetAttribute(latent_tc_kernel<NB, HS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  cudaError_t e = cudaFuncSetAttribute(latent_tc_kernel<NB, HS, SHARED>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   if (e != cudaSuccess) {
     set_error("latent_attn: cudaFuncSetAttribute: %s", cudaGetErrorString(e));
     return DGPT_E_CUDA;
   }
-  launch_dep(latent_tc_kernel<NB, HS>, dim3(grid), dim3(kLtThreads), smem, st, mq, mc, p);
+  launch_dep(latent_tc_kernel<NB, HS, SHARED>, dim3(grid), dim3(kLtThreads), smem, st, mq, mc, p);
   return launch_status("latent_attn");
 }
 
@@ -625,11 +639,16 @@ int latent_tc_launch(const LatentArgs& a, const dgpt_kv_layout& kv, cudaStream_t
   }
   const size_t smem = sh.bytes(p.n_units);
   const int grid = p.n_items < per_sm * sms ? p.n_items : per_sm * sms;
-  if (p.per <= 4) return lt_launch<1, 4>(mq, mc, p, grid, smem, st);
-  if (p.per <= 8) return lt_launch<1, 8>(mq, mc, p, grid, smem, st);
-  if (N == 16) return lt_launch<1, 16>(mq, mc, p, grid, smem, st);
-  if (N == 32) return lt_launch<2, 32>(mq, mc, p, grid, smem, st);
-  return lt_launch<4, 64>(mq, mc, p, grid, smem, st);
+  if (a.v_col == 0) {
+    if (N == 16) return lt_launch<1, 16, true>(mq, mc, p, grid, smem, st);
+    if (N == 32) return lt_launch<2, 32, true>(mq, mc, p, grid, smem, st);
+    return lt_launch<4, 64, true>(mq, mc, p, grid, smem, st);
+  }
+  if (p.per <= 4) return lt_launch<1, 4, false>(mq, mc, p, grid, smem, st);
+  if (p.per <= 8) return lt_launch<1, 8, false>(mq, mc, p, grid, smem, st);
+  if (N == 16) return lt_launch<1, 16, false>(mq, mc, p, grid, smem, st);
+  if (N == 32) return lt_launch<2, 32, false>(mq, mc, p, grid, smem, st);
+  return lt_launch<4, 64, false>(mq, mc, p, grid, smem, st);
 }
 
 }  // namespace dgpt
