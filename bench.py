@@ -929,6 +929,8 @@ def kernel_case(name: str, iters: int = 8) -> None:
     linear:      first feed-forward GEMM of a config-4 decode step with the SwiGLU epilogue.
     latent_attn: decode attention on cached latents, 296 rows x 16 heads x 1024 keys of 256 numbers.
     fmha_window: prefill attention with a window of 1024, 8192 tokens, 16 heads of 128.
+    grouped_attn: grouped-query decode attention, 256 rows, 16 heads on 4 key/value heads of 128, window 1024 of 2048 keys.
+    retention:   chunked retention, 8 sequences of 2048 tokens, 16 heads of 128 x 128.
     Prints one JSON line with the CUDA-event time per launch and the achieved rate.
     """
     from diff_gpt_b200 import ops
@@ -1041,6 +1043,42 @@ def kernel_case(name: str, iters: int = 8) -> None:
 
         work = 4 * D * H * (T * W - W * (W - 1) // 2)
         unit, peak = "TFLOP/s", pk["bf16_tflops"]
+    elif name == "grouped_attn":
+        # one decode step of a grouped-query layer: 256 rows in 64-token pages, 4 kept first tokens (2.1 GB of cache, 0.54 read)
+        R, H, G, D, W, pt, n = 256, 16, 4, 128, 1024, 64, 2048
+        width = 2 * G * D
+        pool = torch.randn((R * n // pt, pt, width), device=dev, dtype=torch.bfloat16, generator=g)
+        table = torch.randperm(R * n // pt, device=dev, generator=g).to(torch.int32).view(R, n // pt)
+        lay = ops.kv_layout(pool, pool, pt * width, 0, pt, table, n_pages=R * n // pt)
+        q = torch.randn((R, H * D), device=dev, dtype=torch.bfloat16, generator=g)
+        o = torch.empty_like(q)
+        zero, n1 = torch.zeros(R, dtype=torch.int32, device=dev), torch.full((R,), n, dtype=torch.int32, device=dev)
+        st = torch.zeros(1, dtype=torch.int32, device=dev)
+
+        def launch():
+            ops.grouped_attn(q, lay, None, zero, n1, None, o, row_width=width, v_col=G * D, n_seq=R, T=1, H=H, G=G, dk=D, dv=D, window=W,
+                             keep_first=4, scale=D**-0.5, status=st)
+
+        work = R * ((W + 4) * width + 2 * H * D) * 2
+        unit, peak = "GB/s", pk["hbm_gbs"]
+    elif name == "retention":
+        # chunked retention of a prefill: q, k, v, gate read and y written once (336 MB)
+        from diff_gpt_b200.model.rope import rotation_table
+
+        B, T, H, D = 8, 2048, 16, 128
+        x = torch.randn((B * T, 4 * H * D), device=dev, dtype=torch.bfloat16, generator=g)
+        y, state = torch.empty((B * T, H * D), device=dev, dtype=torch.bfloat16), torch.empty(B, H, D, D, device=dev)
+        decay = torch.tensor([1 - 2.0 ** (-5 - 6 * j / (H - 1)) for j in range(H)], device=dev)
+        ws = torch.empty(ops.retention_workspace_bytes(B, T, H, D, D) // 4, device=dev)
+        tab, zero = rotation_table(1e4, D, T, dev), torch.zeros(B, dtype=torch.int32, device=dev)
+        st = torch.zeros(1, dtype=torch.int32, device=dev)
+
+        def launch():
+            ops.retention(x, (0, H * D, 2 * H * D, 3 * H * D), tab, zero, None, decay, 0.96, D**-0.5, None, state, 1e-6, y, ws, n_seq=B, T=T,
+                          dim=D, vdim=D, status=st)
+
+        work = B * T * H * 5 * D * 2
+        unit, peak = "GB/s", pk["hbm_gbs"]
     elif name == "sample":
         R, V = TRAJECTORIES, CFG4["vocab_size"]
         logits = (torch.randn((R, V), device=dev, generator=g) * 0.05).to(torch.bfloat16)  # near-flat, as at random init
@@ -1463,7 +1501,7 @@ def run_design(args) -> None:
 
 def main() -> None:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--kernel-case", default=None, choices=["decode_attn", "fmha", "fmha_long", "fmha_pair", "sample", "depthmix", "fmha_prefix", "linear", "latent_attn", "fmha_window"],
+    ap.add_argument("--kernel-case", default=None, choices=["decode_attn", "fmha", "fmha_long", "fmha_pair", "sample", "depthmix", "fmha_prefix", "linear", "latent_attn", "fmha_window", "grouped_attn", "retention"],
                     help="run one kernel alone on a small case (for ncu) and exit")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=3)

@@ -64,14 +64,15 @@ __device__ __forceinline__ float head_gate(const void* hgate, long long rs, long
 __device__ __forceinline__ int window_first_tile(int window, int first_q, int tile) {
   return window > 0 ? max(0, first_q - window + 1) / tile : 0;
 }
-// Key tiles ahead of that one that hold kept first keys.  A query tile visits tiles [0, n_kept) and then those from
-// `tile0` on: its j-th tile is tile_of(j).
+// Key tiles ahead of that one that hold kept first keys.  A query tile visits the n_window tiles from `tile0` on and then
+// tiles [0, n_kept): its j-th tile is tile_of(j).  (The kept ones last: by then the running maximum is settled, and a tile of
+// which a few keys are seen seldom moves it.)
 __device__ __forceinline__ int kept_tiles(int keep_first, int tile0, int tile) {
   return min(tile0, (keep_first + tile - 1) / tile);
 }
 template <bool KEPT>
-__device__ __forceinline__ int tile_of(int j, int n_kept, int tile0) {
-  return KEPT && j < n_kept ? j : tile0 + (j - n_kept);
+__device__ __forceinline__ int tile_of(int j, int n_window, int tile0) {
+  return KEPT && j >= n_window ? j - n_window : tile0 + j;
 }
 
 // warp-level kernel (fmha_simt.cu)

@@ -59,10 +59,10 @@ fmha_simt_kernel(const T* __restrict__ q, long long q_bs, long long q_rs, KvView
   const T* kbase = static_cast<const T*>(kv.k);
   const T* vbase = static_cast<const T*>(kv.v);
 
-  const int tile0 = window_first_tile(window, q_offset + q0, kSimtBN), n_kept = kept_tiles(keep_first, tile0, kSimtBN);
-  for (int tile = 0;; ++tile) {
-    const int j0 = tile_of<true>(tile, n_kept, tile0) * kSimtBN;
-    if (j0 >= kmax) break;
+  const int tile0 = window_first_tile(window, q_offset + q0, kSimtBN), n_window = max(0, (kmax + kSimtBN - 1) / kSimtBN - tile0);
+  const int n_tiles = n_window + kept_tiles(keep_first, tile0, kSimtBN);
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    const int j0 = tile_of<true>(tile, n_window, tile0) * kSimtBN;
     __syncthreads();
     constexpr int VPR = D / VEC;  // 16-byte vectors per key row
     for (int idx = tid; idx < kSimtBN * VPR; idx += 128) {
@@ -256,8 +256,9 @@ static int fmha_sliding(const char* what, const void* q, int64_t q_batch_stride,
   a.hgate = gate; a.hgate_rs = gate_row_stride;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   // The persistent kernel from 1024 keys on, as for full attention, unless the window leaves a query tile only a few key
-  // tiles (16 heads, 8192 tokens: window 128 39 against 46 us, 512 level, 1024 126 against 107 us).
-  a.two_cta = impl == 3 || (impl == 0 && (n_keys < 1024 || (window > 0 && window <= 512)));
+  // tiles (16 heads, 8192 tokens: window 128 39 against 46 us, 512 level, 1024 126 against 107 us; with kept first keys the
+  // persistent one is ahead at 256 and 512 too).
+  a.two_cta = impl == 3 || (impl == 0 && (n_keys < 1024 || (window > 0 && window <= 512 && keep_first == 0)));
   const bool tc_ok = fmha_tc_supported(a, kv);
   if (impl >= 2 && !tc_ok) {
     set_error("%s: the tensor-core kernels do not cover dtype %d, head_dim %d with this layout", what, dtype, D);

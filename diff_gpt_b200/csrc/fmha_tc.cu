@@ -92,12 +92,12 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
   const int klen = p.kv_len ? p.kv_len[b] : p.kv_len_all;
   const int kmax = p.causal ? min(klen, p.q_offset + min(q0 + kBM, p.Tq)) : klen;
   const int tile0 = window_first_tile(p.window, p.q_offset + q0, kBN);
-  const int n_kept = KEPT ? kept_tiles(p.keep_first, tile0, kBN) : 0, kvh = p.kv_div == 1 ? h : h / p.kv_div;
-  const int n_tiles = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0) + n_kept;
+  const int n_window = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - tile0), kvh = p.kv_div == 1 ? h : h / p.kv_div;
+  const int n_tiles = n_window + (KEPT ? kept_tiles(p.keep_first, tile0, kBN) : 0);
 
   // Issue the TMA loads of key/value tile j (thread 0 only).  One box per page and per 64-wide half.
   auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t bar, int j) {
-    const int t0 = tile_of<KEPT>(j, n_kept, tile0) * kBN;
+    const int t0 = tile_of<KEPT>(j, n_window, tile0) * kBN;
     if (pt >= kBN) {
       const int lp = t0 / pt, in = t0 - lp * pt;
       const int pg = p.page_table ? p.page_table[(long long)b * p.max_pages + lp] : b;
@@ -131,7 +131,7 @@ fmha_tc_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant__ C
 
   for (int j = 0; j < n_tiles; ++j) {
     const uint32_t par = (uint32_t)(j & 1);
-    const int t0 = tile_of<KEPT>(j, n_kept, tile0) * kBN;
+    const int t0 = tile_of<KEPT>(j, n_window, tile0) * kBN;
     // ---- S = Q K^T ----
     if (tid == 0) {
       bool ok = true;

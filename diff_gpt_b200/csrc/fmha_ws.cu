@@ -35,7 +35,7 @@ constexpr int kWsThreads = 320;  // 8 softmax warps, the MMA issuer's warp, the 
 constexpr uint32_t kWsTmemCols = 512;
 
 struct WsItem {
-  int b, h, kvh, q0, klen, tile0, n_kept, n;  // n = key tiles: n_kept of kept first keys, then those from tile0 on (see tile_of)
+  int b, h, kvh, q0, klen, tile0, n_window, n;  // n = key tiles: n_window from tile0 on, then those of kept first keys (see tile_of)
 };
 
 template <bool KEPT>
@@ -48,8 +48,8 @@ __device__ __forceinline__ WsItem ws_item(const TcParams& p, int bh, int qt) {
   it.klen = p.kv_len ? p.kv_len[it.b] : p.kv_len_all;
   const int kmax = p.causal ? min(it.klen, p.q_offset + min(it.q0 + kBM, p.Tq)) : it.klen;
   it.tile0 = window_first_tile(p.window, p.q_offset + it.q0, kBN);
-  it.n_kept = KEPT ? kept_tiles(p.keep_first, it.tile0, kBN) : 0;
-  it.n = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0) + it.n_kept;
+  it.n_window = max(0, (kmax > 0 ? (kmax + kBN - 1) / kBN : 0) - it.tile0);
+  it.n = it.n_window + (KEPT ? kept_tiles(p.keep_first, it.tile0, kBN) : 0);
   return it;
 }
 
@@ -123,7 +123,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
         const WsItem it = ws_item<KEPT>(p, bh, qt);
         if (it.n == 0) continue;
         auto load_kv = [&](const CUtensorMap* map, uint32_t dst, uint32_t full, int j) {
-          const int t0 = tile_of<KEPT>(j, it.n_kept, it.tile0) * kBN, kvh = it.kvh;
+          const int t0 = tile_of<KEPT>(j, it.n_window, it.tile0) * kBN, kvh = it.kvh;
           if (pt >= kBN) {
             const int lp = t0 / pt, in = t0 - lp * pt;
             const int pg = p.page_table ? p.page_table[(long long)it.b * p.max_pages + lp] : it.b;
@@ -269,7 +269,7 @@ fmha_tc_ws_kernel(const __grid_constant__ CUtensorMap mq, const __grid_constant_
       float m = -INFINITY, l = 0.f;
       for (int j = 0; j < n_tiles; ++j) {
         const unsigned g = g0 + (unsigned)j, buf = g & 1u, ph = (g >> 1) & 1u;
-        const int t0 = tile_of<KEPT>(j, it.n_kept, it.tile0) * kBN;
+        const int t0 = tile_of<KEPT>(j, it.n_window, it.tile0) * kBN;
         // exits are taken by whole warps (the vote makes the decision uniform), never by single lanes
         if (!__all_sync(0xffffffffu, wait_or_abort(bar_s0 + 8 * buf, ph, abort_flag, 23))) {
           fail = true;

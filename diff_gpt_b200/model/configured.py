@@ -11,8 +11,10 @@ import torch
 import torch.nn as nn
 import torch.nn.functional as F
 
-from .gpt import DeviceModel
+from .gpt import DeviceModel, _sm_count
 from .kv_cache import RowCache
+
+FUSED_FF_MIN_ROWS = 256  # rows from which the up projection runs on the library's GEMM with the activation fused
 
 
 @contextlib.contextmanager
@@ -29,6 +31,14 @@ def fp32_reductions():
 
 def round_up(n: int, m: int) -> int:
     return -(-n // m) * m
+
+
+def pick_latent_splits(rows: int, head_groups: int, keys: int) -> int:
+    """Attention over cached rows: CTAs per row along the keys: enough that every multiprocessor has one, each with a 128-key tile at least."""
+    ctas = max(1, rows * head_groups)
+    if ctas >= _sm_count() or keys <= 128:
+        return 1
+    return max(1, min(_sm_count() // ctas, -(-keys // 128), 64))
 
 
 class ConfiguredModel(DeviceModel):

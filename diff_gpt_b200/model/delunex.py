@@ -33,13 +33,11 @@ import torch.nn.functional as F
 
 from .. import ops
 from .._lib import region
-from .configured import ConfiguredModel, fp32_reductions, round_up
-from .gpt import _sm_count
+from .configured import FUSED_FF_MIN_ROWS, ConfiguredModel, fp32_reductions, pick_latent_splits, round_up
 from .kv_cache import LatentCache, PagedLatentCache
 
 EXPAND_MIN_TOKENS = 32  # query tokens per sequence from which keys and values are expanded
 EXPAND_HEAD_DIMS = (32, 64, 128)  # head sizes of the tensor-core attention kernels; smaller heads are padded with zeros
-FUSED_FF_MIN_ROWS = 256  # rows from which the up projection runs on the library's GEMM with the activation fused
 
 
 # ---- configuration --------------------------------------------------------------------
@@ -196,14 +194,6 @@ class LatentBinding:
     conv_in: torch.Tensor | None = None  # [n_layer, n_seq, taps - 1, C]
     conv_out: torch.Tensor | None = None
     fmha_impl: int = 0
-
-
-def pick_latent_splits(rows: int, head_groups: int, keys: int) -> int:
-    """CTAs per row along the keys: enough that every multiprocessor has one, each with a 128-key tile at least."""
-    ctas = max(1, rows * head_groups)
-    if ctas >= _sm_count() or keys <= 128:
-        return 1
-    return max(1, min(_sm_count() // ctas, -(-keys // 128), 64))
 
 
 class DelunexPlan:

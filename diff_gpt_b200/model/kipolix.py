@@ -37,8 +37,7 @@ import torch.nn.functional as F
 
 from .. import ops
 from .._lib import region
-from .configured import ConfiguredModel, fp32_reductions, round_up
-from .delunex import FUSED_FF_MIN_ROWS, pick_latent_splits
+from .configured import FUSED_FF_MIN_ROWS, ConfiguredModel, fp32_reductions, pick_latent_splits, round_up
 from .kv_cache import PagedRowCache, RowCache, StateSpec
 from .rope import rotation_table
 
