@@ -10,8 +10,8 @@
 // bits; v is bf16 to begin with.  A chunk is shorter than 128 tokens where decay^(2n) would leave fp32's range.
 //
 // One CTA per (sequence, head, 128 value columns, segment of the tokens).  Few heads leave most SMs idle, so a long sequence
-// is cut into segments: retention_state_kernel forms each segment's own contribution to the state, retention_tc_kernel
-// starts each segment from the decayed sum of those before it.
+// is cut into segments: retention_state_kernel forms each segment's own contribution to the state, retention_prefix_kernel
+// adds them up to the state behind each segment, and retention_tc_kernel starts every segment from there.
 //   warps 0-15      rotate, split and write q^, k^ of a chunk into swizzled shared memory (v goes there by cp.async); A -> P;
 //                   state -> shared memory; head norm, output gate and store.  Where every dimension is rotated the next
 //                   chunk's q and k are fetched into registers while the products of this one run
@@ -305,21 +305,20 @@ __global__ void __launch_bounds__(kRtThreads, 1) retention_state_kernel(const Rt
   bool fail = false;
   int tile = 0;
   RtRows<false, ND> next;
-  if (PLAIN && warp < 16) next.load(a, hd, t_begin, min(kRtChunk, t_end - t_begin), tid);
+  // v of a tile comes by cp.async while the tile before is finished, k through registers
+  auto fetch = [&](int t0, int b) {
+    const int n = min(kRtChunk, t_end - t0);
+    rt_load_v<NV>(a, hd, t0, n, smem_u32(smem + b * buf_bytes + 2 * ND * kRtBlock), tid);
+    if (PLAIN) next.load(a, hd, t0, n, tid);
+    rt_prefetch<false, ND, NV>(a, hd, t0 + kRtChunk, max(0, min(kRtChunk, t_end - t0 - kRtChunk)), tid);
+  };
+  if (warp < 16) fetch(t_begin, 0);
   for (int t0 = t_begin; t0 < t_end; t0 += kRtChunk, ++tile) {
     const int n = min(kRtChunk, t_end - t0), b = tile & 1;
     uint8_t* sK = smem + b * buf_bytes;
-    uint8_t* sV = sK + 2 * ND * kRtBlock;
     if (warp < 16) {
-      if (tile >= 2 && !wait_or_abort(bar + 8 * b, ((tile >> 1) - 1) & 1u, abort_flag, 63)) fail = true;  // the buffer has been read
-      rt_load_v<NV>(a, hd, t0, n, smem_u32(sV), tid);
-      rt_prefetch<false, ND, NV>(a, hd, t0 + 2 * kRtChunk, max(0, min(kRtChunk, t_end - t0 - 2 * kRtChunk)), tid);
-      if (PLAIN) {
-        next.store(a, hd, t0, n, t_end - 1 - t0, l2, pw, sK, nullptr, lo_off, tid);
-        if (t0 + kRtChunk < t_end) next.load(a, hd, t0 + kRtChunk, min(kRtChunk, t_end - t0 - kRtChunk), tid);
-      } else {
-        rt_build_any<false>(a, hd, t0, n, t_end - 1 - t0, l2, sK, nullptr, ND, tid);
-      }
+      if (PLAIN) next.store(a, hd, t0, n, t_end - 1 - t0, l2, pw, sK, nullptr, lo_off, tid);
+      else rt_build_any<false>(a, hd, t0, n, t_end - 1 - t0, l2, sK, nullptr, ND, tid);
       rt_cp_wait();
       fence_async_smem();
     }
@@ -329,12 +328,17 @@ __global__ void __launch_bounds__(kRtThreads, 1) retention_state_kernel(const Rt
     }
     if (warp == 16 && lane == 0) {
       tc_fence_after();
-      const uint32_t aK = smem_u32(sK), aV = smem_u32(sV);
+      const uint32_t aK = smem_u32(sK), aV = aK + 2 * ND * kRtBlock;
       umma_ss8<128, 512, 128, 512>(tmem, dM + (aK >> 4), dM + (aV >> 4), idesc_s, tile > 0 ? 1u : 0u);
       umma_ss8<128, 512, 128, 512>(tmem, dM + ((aK + lo_off) >> 4), dM + (aV >> 4), idesc_s, 1u);
       umma_commit(bar + 8 * b);
     }
+    if (warp < 16 && t0 + kRtChunk < t_end) {
+      if (tile >= 1 && !wait_or_abort(bar + 8 * (b ^ 1), ((tile - 1) >> 1) & 1u, abort_flag, 63)) fail = true;  // the other buffer has been read
+      fetch(t0 + kRtChunk, b ^ 1);
+    }
   }
+  rt_cp_wait();
   // the last two tiles' products (the others were waited for)
   for (int t = max(0, tile - 2); t < tile; ++t)
     if (!wait_or_abort(bar + 8 * (t & 1), (t >> 1) & 1u, abort_flag, 64)) fail = true;
@@ -357,6 +361,32 @@ __global__ void __launch_bounds__(kRtThreads, 1) retention_state_kernel(const Rt
   tc_fence_before();
   __syncthreads();
   if (warp == 0) tmem_dealloc(tmem, 128);
+}
+
+// ---- from what each segment adds to the state behind each segment, in place ---------------------------------------
+// Thread per four numbers of a head's state; carried in: a.state_in (or zeros).
+__global__ void __launch_bounds__(256) retention_prefix_kernel(const RtParams p, long long per_head4) {
+  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
+  if (i >= per_head4) return;
+  const int sh = blockIdx.y;  // sequence * H + head
+  const float f = rt_pow(log2f(p.a.decay[sh % p.a.H]), p.seg_len);
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  if (p.a.state_in) acc = reinterpret_cast<const float4*>(p.a.state_in)[sh * per_head4 + i];
+  float4* seg = reinterpret_cast<float4*>(p.seg_state) + (long long)sh * (p.n_seg - 1) * per_head4 + i;
+  const int n = p.n_seg - 1;  // every segment but the last is full
+  for (int r0 = 0; r0 < n; r0 += 8) {
+    float4 u[8];
+#pragma unroll
+    for (int r = 0; r < 8; ++r)
+      if (r0 + r < n) u[r] = seg[(r0 + r) * per_head4];
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      if (r0 + r < n) {
+        acc = make_float4(fmaf(f, acc.x, u[r].x), fmaf(f, acc.y, u[r].y), fmaf(f, acc.z, u[r].z), fmaf(f, acc.w, u[r].w));
+        seg[(r0 + r) * per_head4] = acc;
+      }
+    }
+  }
 }
 
 // ---- the chunks -----------------------------------------------------------------------------------
@@ -477,19 +507,14 @@ __global__ void __launch_bounds__(kRtThreads, 1) retention_tc_kernel(const RtPar
 #pragma unroll
       for (int i = 0; i < 32; ++i) v[i] = 0.f;
       if (row < a.dim) {
-        for (int r = -1; r < seg; ++r) {  // -1: the state carried in
-          if (r < 0 && a.state_in == nullptr) continue;
-          const float f = rt_pow(l2, t_begin - (r + 1) * p.seg_len);
-          const float* src = r < 0 ? a.state_in + st0 : p.seg_state + sg0 + (long long)r * a.dim * a.vdim;
+        const float* src = seg > 0 ? p.seg_state + sg0 + (long long)(seg - 1) * a.dim * a.vdim : a.state_in ? a.state_in + st0 : nullptr;
+        if (src) {
           src += (long long)row * a.vdim + c * 32;
 #pragma unroll
           for (int i = 0; i < 32; i += 4) {
             if (c * 32 + i < ne) {  // ne is a multiple of 8
               const float4 t = *reinterpret_cast<const float4*>(src + i);
-              v[i] = fmaf(f, t.x, v[i]);
-              v[i + 1] = fmaf(f, t.y, v[i + 1]);
-              v[i + 2] = fmaf(f, t.z, v[i + 2]);
-              v[i + 3] = fmaf(f, t.w, v[i + 3]);
+              v[i] = t.x; v[i + 1] = t.y; v[i + 2] = t.z; v[i + 3] = t.w;
             }
           }
         }
@@ -685,6 +710,9 @@ static int rt_launch(const RtParams& p, cudaStream_t st) {
   if (p.n_seg > 1) {
     retention_state_kernel<ND, NV, PLAIN><<<heads * (p.n_seg - 1), kRtThreads, rt_smem_state(ND, NV), st>>>(p);
     if (int e = launch_status("retention_state")) return e;
+    const long long per_head4 = (long long)p.a.dim * p.a.vdim / 4;
+    retention_prefix_kernel<<<dim3((unsigned)((per_head4 + 255) / 256), (unsigned)(p.a.n_seq * p.a.H)), 256, 0, st>>>(p, per_head4);
+    if (int e = launch_status("retention_prefix")) return e;
   }
   retention_tc_kernel<ND, NV, PLAIN><<<heads * p.n_seg, kRtThreads, rt_smem_main(ND, NV), st>>>(p);
   return launch_status("retention_tc");
