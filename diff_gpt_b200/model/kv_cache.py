@@ -10,6 +10,10 @@ write its dense (L, 2, B, H, T, D) tensor in place through `layer_layout`.
 the prompt (the reference's `prefill` broadcast, kv_cache.py:79): K/V live in
 fixed-size pages, every trajectory of a series points at the SAME prompt pages,
 and each trajectory owns a contiguous run of pages for the tokens it generates.
+
+`RowCache` (requests fed step by step) and `PagedRowCache` (the engine) serve the models that are built from a
+configuration: one row of numbers per token and layer run, bounded by the windows, and the per-sequence state
+(`SeqState`) that such models carry beside it.
 """
 
 from __future__ import annotations
